@@ -140,7 +140,7 @@ sdpa_decode_kernel(SdpaParams p) {
     constexpr int TP = AttnTile<DT, HD>::TP;               // KV positions per staged tile
     constexpr uint32_t ROWB = HD * esz;                      // bytes of one K (or V) row
     constexpr uint32_t TILEB = TP * ROWB;                    // bytes of one K (or V) tile
-    // K/V tiles are contiguous in the [n_kv, max_seq, hd] cache, so one cp.async.bulk (TMA, UBLKCP) per
+    // K/V tiles are contiguous in the [n_kv, max_seq, hd] cache, so one cp.async.bulk (TMA) per
     // tensor stages a whole tile in shared memory; kAttnStages tiles are in flight per CTA (>= 64 KB per
     // SM with two resident CTAs), decoupling the HBM latency from the softmax arithmetic.
     extern __shared__ __align__(128) unsigned char kv_smem[];
@@ -411,14 +411,14 @@ struct RopeSdpaParams {
     long qkv_stride, out_stride, cache_stride;     // elements between consecutive sequences
 };
 // ---------------------------------------------------------------------------------------------------------------
-// The score and P.V products run on the tensor cores (mma.sync m16n8k16, SASS HMMA)
-// and the K/V tiles fetched by tensor-map TMA (cp.async.bulk.tensor.4d, SWIZZLE_128B, SASS UTMALDG) so that ldmatrix
+// The score and P.V products run on the tensor cores (mma.sync m16n8k16)
+// and the K/V tiles fetched by tensor-map TMA (cp.async.bulk.tensor.4d, SWIZZLE_128B) so that ldmatrix
 // reads them without bank conflicts.  Decode attention is HBM / latency bound; the CUDA-core loop of round 1 spent 450
 // issue slots per warp per 64 positions (unpacking V, 15 shuffles of the score reduce-scatter), which bounded the long
 // contexts and the multi-sequence batches.  Here a warp owns 16 positions of a 64-position tile:
-//     S[8 heads (+8 zero rows), 16 pos]  = Q[16, 128] . K^T      16 HMMA, B fragments by ldmatrix from the swizzled tile
+//     S[8 heads (+8 zero rows), 16 pos]  = Q[16, 128] . K^T      16 MMAs, B fragments by ldmatrix from the swizzled tile
 //     online softmax on the 4 scores a thread holds (row = lane / 4), quad shuffles only
-//     O[16, 128] += P[16, 16] . V[16, 128]                       16 HMMA, V fragments by ldmatrix.trans
+//     O[16, 128] += P[16, 16] . V[16, 128]                       16 MMAs, V fragments by ldmatrix.trans
 // The probabilities go to the tensor cores as TWO bf16 terms, p = hi + lo, hi in rows 0..7 and lo in rows 8..15 of the
 // A fragment (the rows the <= 8 query heads leave empty), so one MMA accumulates both and O = O[0..7] + O[8..15] carries
 // 16 bits of p: the products q.k are exact and p.v is as accurate as the f32 loop it replaces.

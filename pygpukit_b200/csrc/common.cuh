@@ -127,7 +127,7 @@ __device__ __forceinline__ uint32_t pack_bf16x2(float lo, float hi) {
 }
 
 // streaming loads: read-only path, do not allocate in L1, evict-first in L2 (weights are
-// touched once per token).  sm_100a has 256-bit global loads (LDG.E.NA.EFL2.256).
+// touched once per token).  sm_100a has 256-bit global loads.
 struct alignas(32) u32x8 { uint32_t v[8]; };
 __device__ __forceinline__ u32x8 ldg_stream256(const void* p) {
     u32x8 r;
@@ -220,7 +220,7 @@ __device__ __forceinline__ float e2m1_to_f32(uint32_t nib) {
 }
 
 
-// ---- mbarrier + TMA bulk copy (cp.async.bulk, SASS UBLKCP): contiguous global -> shared, completion
+// ---- mbarrier + TMA bulk copy (cp.async.bulk): contiguous global -> shared, completion
 // counted in bytes on an mbarrier.  No tensor map needed for 1-D tiles.
 __device__ __forceinline__ uint32_t smem_u32(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
 __device__ __forceinline__ void mbar_init(uint64_t* bar, int count) {

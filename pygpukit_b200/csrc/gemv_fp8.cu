@@ -8,7 +8,7 @@
 // Design (HBM-bound; see DESIGN.md "gemv_fp8"):
 //   * one wave: every warp of the grid is resident at once and owns `rho` consecutive
 //     weight rows; the host picks (warps/CTA, CTAs/SM) so that N / (rho * warps) ~ 1.
-//   * weights stream with 256-bit ld.global.nc.L1::no_allocate.L2::evict_first loads (LDG.E.NA.EFL2.256), four
+//   * weights stream with 256-bit ld.global.nc.L1::no_allocate.L2::evict_first loads, four
 //     256-bit loads in flight per lane; they are read ONCE for all M activation rows.
 //   * dequantisation in registers: F2FP.F16.E4M3.UNPACK_B turns two codes into an exact
 //     f16x2; the product with the activation is the mixed-precision FHFMA

@@ -8,7 +8,7 @@
 // Design (HBM-bound; DESIGN.md "step program"):
 //   * grid = one CTA per SM, 16 consumer warps + 1 producer warp.  The producer walks the SAME op list as the
 //     consumers and streams every byte the CTA will need (weight rows, K/V tiles) into a ring of 8 KB shared-memory
-//     slots with cp.async.bulk (TMA, SASS UBLKCP) completing on per-slot mbarriers.  Weights and old KV rows are
+//     slots with cp.async.bulk (TMA) completing on per-slot mbarriers.  Weights and old KV rows are
 //     constants of the step, so the producer never waits for a grid barrier: while the consumers synchronise and
 //     re-stage the activation vector (~2 us per op boundary) the ring keeps filling (up to ~190 KB per SM = 28 MB
 //     in flight on the GPU), and the HBM stream does not stop at op boundaries.

@@ -1,5 +1,5 @@
 // tc_common.cuh -- tcgen05 / TMEM primitives shared by the tensor-core skinny GEMMs (gemm_tc.cu: FP8 weights,
-// gemm_tc_nvf4.cu: NVF4 weights).  Raw PTX; SASS shows UTCHMMA (tcgen05.mma), LDTM (tcgen05.ld), UTCBAR (commit).
+// gemm_tc_nvf4.cu: NVF4 weights).  Hand-written PTX: tcgen05.mma, tcgen05.ld, tcgen05.commit.
 #pragma once
 #include "common.cuh"
 
