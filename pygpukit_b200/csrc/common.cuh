@@ -118,8 +118,8 @@ __device__ __forceinline__ uint16_t hadd_bf16_bits(float a, uint16_t b_bits) {
     __nv_bfloat16 r = __hadd(__float2bfloat16_rn(a), __ushort_as_bfloat16(b_bits));
     return __bfloat16_as_ushort(r);
 }
-// two f32 -> packed bf16x2 with ONE full-rate instruction (cvt.rn.bf16x2.f32 = F2FP.BF16.F32.PACK_AB); the
-// scalar F2F.BF16.F32 runs on the quarter-rate conversion pipe
+// two f32 -> packed bf16x2 with ONE full-rate instruction (cvt.rn.bf16x2.f32); the
+// scalar conversion runs on the quarter-rate conversion pipe
 __device__ __forceinline__ uint32_t pack_bf16x2(float lo, float hi) {
     uint32_t r;
     asm("cvt.rn.bf16x2.f32 %0, %1, %2;" : "=r"(r) : "f"(hi), "f"(lo));
@@ -183,7 +183,7 @@ __device__ __forceinline__ void fhfma_f16_hl(float& acc, uint32_t a, uint32_t b)
         " fma.rn.f32.f16 %0, ah, bl, %0;}" : "+f"(acc) : "r"(a), "r"(b));
 }
 
-// two e4m3 bytes (low / high half of a 32-bit word) -> f16x2 (exact).  F2FP.F16.E4M3.UNPACK_B
+// two e4m3 bytes (low / high half of a 32-bit word) -> f16x2 (exact)
 __device__ __forceinline__ uint32_t e4m3x2_to_f16x2_lo(uint32_t w) {
     uint32_t r;
     asm("{.reg .b16 lo, hi; mov.b32 {lo, hi}, %1; cvt.rn.f16x2.e4m3x2 %0, lo;}" : "=r"(r) : "r"(w));

@@ -12,9 +12,9 @@
 //     M = 128 -> one TMEM lane per weight row) and the batch is the MMA's N (16 / 32 / 64 f32 TMEM columns);
 //     split-K over gridDim.y fills the 148 SMs when N/128 tiles are too few.
 //   * per 128-wide k block (= one FP8 scale block; the 128-row tile lies inside one scale row, so the CTA sees
-//     ONE scale per k block): 16 KB of E4M3 codes stream global -> shared memory with cp.async (LDGSTS, a ring of
+//     ONE scale per k block): 16 KB of E4M3 codes stream global -> shared memory with cp.async (a ring of
 //     four raw blocks = 64 KB in flight per SM, requested before the dependency wait), are converted exactly to BF16
-//     (F2FP.F16.E4M3.UNPACK_B -> f32 -> BF16x2 pack; E4M3 fits BF16) and stored to shared memory in the
+//     (cvt e4m3x2 -> f16x2 -> f32 -> BF16x2 pack; E4M3 fits BF16) and stored to shared memory in the
 //     canonical no-swizzle K-major core-matrix layout; the [M,128] activation slab is multiplied by the block
 //     scale in f32 and split into TWO BF16 terms, hi = bf16(a*s) and lo = bf16(a*s - hi), stored in the same
 //     layout: with exact BF16 weights the two MMAs reproduce the f32 product a*s*w to ~2^-17, i.e. the
@@ -91,7 +91,7 @@ gemm_fp8_tc_kernel(TcParams p) {
         mbar_fence_init();
     }
 
-    // ---- raw rings (cp.async / LDGSTS): global -> shared in FULL 128-byte lines (8 lanes per weight row, 16 lanes
+    // ---- raw rings (cp.async): global -> shared in FULL 128-byte lines (8 lanes per weight row, 16 lanes
     // per activation row), stored row-major with the 16-byte pieces of a row XOR-swizzled by (row & 7) so that
     // both the line-wise copy and the core-matrix-wise read-back (8 rows x one piece per quarter warp) are
     // bank-conflict free.  Weights never depend on the previous kernel: their first kTcRaw blocks are requested

@@ -19,7 +19,7 @@
 //     the batch is the MMA N (16 / 32 / 64 TMEM columns).
 //   * per 128-wide k block: 64 byte rows x 128 B of nibbles + 4 x 128 B of scales stream global -> shared memory with
 //     cp.async in full 128-byte lines (ring of raw blocks, requested before the dependency wait), thread (k chunk c,
-//     column quad) gathers the four bytes of a column with PRMT, F2FP.F16.E2M1.UNPACK_B -> HMUL2 by the scale (exact
+//     column quad) gathers the four bytes of a column with byte permutes, cvt e2m1x2 -> f16x2, multiplied by the scale (exact
 //     in F16) -> BF16x2, and stores the 16-byte k chunk into the canonical no-swizzle K-major core-matrix layout;
 //     fence.proxy.async; a dedicated warp issues the 8 MMAs of the block and commits to the stage's mbarrier.
 #include "common.cuh"

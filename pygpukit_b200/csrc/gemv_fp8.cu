@@ -10,7 +10,7 @@
 //     weight rows; the host picks (warps/CTA, CTAs/SM) so that N / (rho * warps) ~ 1.
 //   * weights stream with 256-bit ld.global.nc.L1::no_allocate.L2::evict_first loads, four
 //     256-bit loads in flight per lane; they are read ONCE for all M activation rows.
-//   * dequantisation in registers: F2FP.F16.E4M3.UNPACK_B turns two codes into an exact
+//   * dequantisation in registers: cvt.rn.f16x2.e4m3x2 turns two codes into an exact
 //     f16x2; the product with the activation is the mixed-precision FHFMA
 //     (fma.rn.f32.f16: exact product, f32 accumulate) -- 1.5 instructions per weight.
 //     Activations are staged once per CTA in shared memory as f16 after an exact

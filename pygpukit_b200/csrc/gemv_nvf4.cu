@@ -14,7 +14,7 @@
 //     and over KS CTAs per 512-column group.  Partial sums meet in shared memory, then in
 //     an f32 workspace that the last-arriving CTA of the group folds in fixed order
 //     (deterministic, no float atomics).
-//   * dequantisation in registers: F2FP.F16.E2M1.UNPACK_B turns one byte into the exact f16
+//   * dequantisation in registers: cvt.rn.f16x2.e2m1x2 turns one byte into the exact f16
 //     pair (even k, odd k); FHFMA (fma.rn.f32.f16) multiplies by the staged f16 activation
 //     with an exact product and f32 accumulation: 1.5 instructions per weight.
 //   * the UE4M3 block scale is decoded with one shift-add and applied once per 32-k block

@@ -101,7 +101,7 @@ def fp8_get_sizes(K: int, N: int) -> tuple[int, int, int]:
 
 
 def w8a16_gemm_init_lut() -> None:
-    """No-op: the B200 kernels decode E4M3 with F2FP, there is no constant-memory LUT to load."""
+    """No-op: the B200 kernels decode E4M3 with a conversion instruction, there is no constant-memory LUT to load."""
 
 
 def w8a16_gemm_sm120(a: GPUArray, b_fp8: GPUArray, b_scale: GPUArray, *, out: GPUArray | None = None) -> GPUArray:
