@@ -128,7 +128,7 @@ int pgk_gemv_nvf4_bf16_ex(const void* A, const void* B_data, const void* B_scale
                           int K, int N, float alpha, const void* bias, const void* residual,
                           void* stream);
 /* Decode batch 5..64 on the tensor cores: E2M1 x UE4M3 has <= 6 significant bits, so the converter warps write EXACT BF16
- * weight tiles (F2FP.E2M1 unpack, HMUL2 by the scale) and one tcgen05.mma.kind::f16 per 16 k computes exact products with
+ * weight tiles (E2M1 conversion, multiply by the scale) and one tcgen05.mma.kind::f16 per 16 k computes exact products with
  * F32 accumulation in TMEM -- the FP32-accumulate class of the GEMV, weights read once for all M rows.  Needs
  * 1 <= M <= 64, K % 128 == 0, N % 128 == 0; pgk_gemv_nvf4_bf16(_ex) dispatch here for M >= 5.  Replaces the per-row use of
  * gemv_nvf4_bf16_kernel (nvf4_kernels.cu:79-233) and the CUTLASS NVF4 GEMM of gemm/w4a16_bf16/sm120/nvf4_cutlass.cu. */
@@ -643,6 +643,56 @@ int pgk_seq_gated_recurrence(int delta, const float* q, int ldq, int q_off, cons
                              int lda, int a_off, const float* beta, int ldb, int b_off, const float* v, int ldv, int v_off,
                              float* out, int ldo, float* state, const int32_t* seqs, int n_seqs, int heads, int qk_heads, int dim,
                              int vdim, void* stream);
+/* pgk_seq_mixer_prep_rot_ex with more optional parts.  pairs: element 2i turns with 2i + 1 (0: i with i + rot_dims / 2).
+ * norm_first: the norm of q / k and its weight come in front of the rotation.  v_inv_freq [vdim / 2]: the values turn too, over
+ * all vdim elements in the same layout, and are stored so.  pool > 0: every block of `pool` consecutive positions of a sequence
+ * also leaves the means of its key and value rows (as stored) in k_pool [pages][kv_heads][pool_rows][dim] and v_pool
+ * [..][vdim], row b - floor(page_index page_size / pool) of the page that holds the block's last position, written by the
+ * position that follows the block (single_token: every sequence brings one token, no second launch). */
+int pgk_seq_mixer_prep_rot_ex2(float* proj, int ld, int tokens, int heads, int kv_heads, int dim, int vdim, int q_off, int k_off,
+                               int v_off, int rot_dims, const double* inv_freq, int norm_mode, const float* q_weight,
+                               const float* k_weight, float eps, const float* q_bias, const float* k_bias, const float* v_bias,
+                               const float* q_mult, int pairs, int norm_first, const double* v_inv_freq, int pool, int pool_rows,
+                               void* k_pool, void* v_pool, int single_token, void* k_cache, void* v_cache, int cache_dtype,
+                               const int32_t* table, int max_pages, int page_size, const int32_t* slot, const int32_t* pos,
+                               void* stream);
+/* pgk_seq_attention_ex2 with pooled blocks (pool > 0, needs a window: beside its window a query at i sees the pooled key and
+ * value of every block that ends at or before i - window, in the same softmax) and outputs turned back by the query's position
+ * (out_inv_freq [vdim / 2], out_pairs as in the preparation) in front of the gate. */
+int pgk_seq_attention_ex3(const float* q, int ldq, int q_off, const float* gate_rows, int ldg, int gate_off, int gate_mode,
+                          float* out, int ldo, const void* k_cache, const void* v_cache, int k_ld, int v_ld, int cache_dtype,
+                          const int32_t* table, int max_pages, int page_size, const int32_t* tiles, int n_tiles,
+                          const float* slopes, const float* slopes2, const float* sinks, int heads, int kv_heads, int dim,
+                          int vdim, int chunk, int window, int keep_first, float scale, float softcap, int weight_mode,
+                          const float* weight_bias, float out_mult, int pool, int pool_rows, const void* k_pool,
+                          const void* v_pool, const double* out_inv_freq, int out_pairs, int splits, float* workspace,
+                          uint32_t* tickets, int single_query, void* stream);
+/* x[t] += rms(base[t] + sum_k weights[t, k] parts[inv[t, k]]) * weight (base may be NULL, top 0: plain rows). */
+int pgk_rms_join_f32(const float* base, const float* parts, const int32_t* inv, const float* weights, int top, const float* weight,
+                     float eps, float* x, int rows, int width, void* stream);
+/* The `top` largest of logits + bias, weights = softmax over the chosen ones; extra >= 0: matrix `extra` with weight 1 as one
+ * more slot of every token (idx / weights / rank then have top + 1 entries per token, counts experts + 1). */
+int pgk_moe_route_logits(const float* logits, int ld, int tokens, int experts, int top, const float* bias, int extra, int32_t* idx,
+                         float* weights, int32_t* rank, int32_t* counts, void* stream);
+/* The matrix memory of xLSTM (seq_mlstm.cu) on rows that hold q, k [heads x dim], v, gate [heads x vdim] and the two log gates'
+ * projections [heads] at the given columns.  State per slot: S [heads][dim][vdim], N [heads][dim], M [heads].
+ * _step: one token per sequence, one launch.  Longer steps: _gates once (gates: pgk_seq_mlstm_gate_floats floats, 8-byte
+ * aligned; updates M), then _chunks over segments of chunks of pgk_seq_mlstm_chunk_tokens tokens (workspace: n_seqs x chunks x
+ * heads x (dim x vdim + dim) floats), then, when vdim > 128, pgk_seq_linear_finish for norm, weight and gate. */
+int pgk_seq_mlstm_chunk_tokens(void);
+size_t pgk_seq_mlstm_gate_floats(int tokens, int heads);
+int pgk_seq_mlstm_step(const float* proj, int ld, int q_off, int k_off, int v_off, int g_off, int i_off, int f_off,
+                       const float* i_bias, const float* f_bias, float cap, float q_scale, const float* weight, float eps, float* out,
+                       int ldo, float* S, float* N, float* M, const int32_t* seqs, int n_seqs, int heads, int dim, int vdim,
+                       void* stream);
+int pgk_seq_mlstm_gates(const float* proj, int ld, int i_off, int f_off, const float* i_bias, const float* f_bias, float cap,
+                        float* M, const int32_t* seqs, int n_seqs, int tokens, int heads, float* gates, void* stream);
+int pgk_seq_mlstm_chunks(const float* proj, int ld, int q_off, int k_off, int v_off, int g_off, int i_off, int f_off,
+                         const float* i_bias, const float* f_bias, float cap, float q_scale, const float* weight, float eps, float* out,
+                         int ldo, float* S, float* N, float* M, const int32_t* seqs, int n_seqs, int tokens, int heads, int dim, int vdim,
+                         const float* gates, int chunk_begin, int chunks, float* workspace, void* stream);
+int pgk_seq_mlstm_fused_finish(int vdim);
+
 /* mixer_prep for layers whose q / k norm runs over the WHOLE projection: per token, q <- (q + q_bias) / rms(all heads x dim
  * of q) * (weight_offset + q_weight) in place (proj[t, 0 ..]), k the same from proj[t, k_off ..] with k_weight into the K
  * pages; the V pages receive k + k_bias as projected (before the norm).  Biases may be NULL; weights are [heads x dim] and

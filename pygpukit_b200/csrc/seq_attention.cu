@@ -15,6 +15,10 @@
 //                softmax denominator once and has no value: the running (max, sum) starts at (sink, 1) instead of
 //                (-inf, 0)), a gate of one number per head, values that are a prefix of the key rows (latent attention:
 //                one cache array, no second staging), and row strides of the cache rows.
+//                Pooled blocks (a window with pool = P): every P consecutive positions also leave ONE key and ONE value row, the
+//                means of theirs, in arrays beside the pages (row b - floor(page PS / P) of the page that holds the block's last
+//                position); a query sees the blocks that end at or before i - window, in the same softmax as its window.
+//                Values may be stored rotated by their position; the heads' outputs are then turned back by the query's.
 //   mixer_prep_all: the form whose q / k norm runs over the WHOLE projection (all heads at once), with projection
 //                biases and values that are the keys before the norm.
 #include "common.cuh"
@@ -85,23 +89,70 @@ struct PrepRotArgs {
     const int* slot; const int* pos;
     const float* qb; const float* kb; const float* vb;      // projection biases [H x D], [G x D], [G x Dv] or NULL
     const float* q_mult;                                     // [H] factor on every query head (a per-head temperature) or NULL
+    int pairs;                                       // 0: element i turns with i + rot_dims / 2; 1: element 2i with 2i + 1
+    int norm_first;                                  // the norm (and its weight) comes before the rotation
+    const double* v_inv_freq;                        // [Dv / 2] or NULL: values turn too, over all Dv elements in the same layout
+    int pool, pool_rows; void* pk; void* pv;         // pool > 0: this launch also pools (one decoded token per sequence)
 };
 
+// The block of `pool` positions that ends right before `pos` (which starts a block) leaves the means of its key or value rows.
+// unit: 0 .. G - 1 keys, G .. 2G - 1 values; one warp.
+template <typename TC>
+__device__ __forceinline__ void pool_block_rows(const PrepRotArgs& a, int pos, int slot, int unit, int lane) {
+    const bool is_v = unit >= a.G;
+    const int g = is_v ? unit - a.G : unit, n = is_v ? a.Dv : a.D, P = a.pool, b = pos / P - 1;
+    const int* tab = a.table + (size_t)slot * a.max_pages;
+    const int lastpg = (pos - 1) / a.PS, row = b - (int)((long long)lastpg * a.PS / P);
+    const TC* src = (const TC*)(is_v ? a.vc : a.kc);
+    TC* dst = (TC*)(is_v ? a.pv : a.pk) + (((size_t)tab[lastpg] * a.G + g) * a.pool_rows + row) * n;
+    const float inv = 1.f / (float)P;
+    for (int d = lane; d < n; d += 32) {
+        float s = 0.f;
+        for (int j = pos - P; j < pos; ++j) s += cload<TC>(src + (((size_t)tab[j / a.PS] * a.G + g) * a.PS + j % a.PS) * n + d);
+        cstore<TC>(dst + d, s * inv);
+    }
+}
+
+// steps that bring several tokens of a sequence: pooling is a launch of its own, behind the one that writes the rows
+template <typename TC>
+__global__ void __launch_bounds__(128) pool_rows_kernel(PrepRotArgs a) {
+    const int t = blockIdx.x, pos = a.pos[t], u = blockIdx.y * 4 + (threadIdx.x >> 5);
+    if (pos == 0 || pos % a.pool || u >= 2 * a.G) return;
+    pool_block_rows<TC>(a, pos, a.slot[t], u, threadIdx.x & 31);
+}
+
 // units: H query heads (rotated and normalised in place), G key heads and G value heads (into the cache); a warp each.
-// Rotation: element i < rot_dims / 2 of a head is paired with element i + rot_dims / 2, angle = position * inv_freq[i].
+// Rotation: element i < rot_dims / 2 of a head is paired with element i + rot_dims / 2 (or element 2i with 2i + 1), angle =
+// position * inv_freq[i].  The norm comes behind the rotation or, with norm_first, in front of it.
 template <typename TC>
 __global__ void __launch_bounds__(128) mixer_prep_rot_kernel(PrepRotArgs a) {
     const int t = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     const int u = blockIdx.y * 4 + warp;
-    if (u >= a.H + 2 * a.G) return;
+    if (u >= a.H + (a.pool > 0 ? 4 : 2) * a.G) return;
     float* row = a.proj + (size_t)t * a.ld;
     const int pos = a.pos[t], slot = a.slot[t];
+    if (u >= a.H + 2 * a.G) {
+        if (pos > 0 && pos % a.pool == 0) pool_block_rows<TC>(a, pos, slot, u - a.H - 2 * a.G, lane);
+        return;
+    }
     const int page = a.table[(size_t)slot * a.max_pages + pos / a.PS], r = pos % a.PS;
     if (u >= a.H + a.G) {
         const int g = u - a.H - a.G;
         const float* v = row + a.v_off + (size_t)g * a.Dv;
         TC* dst = (TC*)a.vc + (((size_t)page * a.G + g) * a.PS + r) * a.Dv;
         const float* vb = a.vb ? a.vb + (size_t)g * a.Dv : nullptr;
+        if (a.v_inv_freq) {
+            const int vh = a.Dv / 2;
+            for (int i = lane; i < vh; i += 32) {
+                const int i0 = a.pairs ? 2 * i : i, i1 = a.pairs ? 2 * i + 1 : i + vh;
+                float sn, cs;
+                rope_angle_sincos(pos, a.v_inv_freq[i], sn, cs);
+                const float p0 = v[i0] + (vb ? vb[i0] : 0.f), p1 = v[i1] + (vb ? vb[i1] : 0.f);
+                cstore<TC>(dst + i0, p0 * cs - p1 * sn);
+                cstore<TC>(dst + i1, p1 * cs + p0 * sn);
+            }
+            return;
+        }
         for (int d = lane; d < a.Dv; d += 32) cstore<TC>(dst + d, v[d] + (vb ? vb[d] : 0.f));
         return;
     }
@@ -112,28 +163,39 @@ __global__ void __launch_bounds__(128) mixer_prep_rot_kernel(PrepRotArgs a) {
     const float qm = (!is_k && a.q_mult) ? a.q_mult[u] : 1.f;
     if (!is_k && a.rot_dims == 0 && a.norm == 0 && !bias && !a.q_mult) return;      // the query stays as projected
     const int half = a.rot_dims / 2;
-    float ss = 0.f;
+    const bool first = a.norm && a.norm_first;
+    const float* w = a.norm == 2 ? (is_k ? a.kw : a.qw) : nullptr;
+    float ss = 0.f, inv = 1.f;
+    if (first) {
+        for (int d = lane; d < a.D; d += 32) {
+            const float v = x[d] + (bias ? bias[d] : 0.f);
+            ss = fmaf(v, v, ss);
+        }
+        inv = 1.f / sqrtf(warp_sum(ss) / (float)a.D + a.eps);
+    }
     for (int i = lane; i < half; i += 32) {
+        const int i0 = a.pairs ? 2 * i : i, i1 = a.pairs ? 2 * i + 1 : i + half;
         float sn, cs;
         rope_angle_sincos(pos, a.inv_freq[i], sn, cs);
-        const float p0 = x[i] + (bias ? bias[i] : 0.f), p1 = x[i + half] + (bias ? bias[i + half] : 0.f);
+        float p0 = x[i0] + (bias ? bias[i0] : 0.f), p1 = x[i1] + (bias ? bias[i1] : 0.f);
+        if (first) { p0 *= inv * (w ? w[i0] : 1.f); p1 *= inv * (w ? w[i1] : 1.f); }
         const float r0 = p0 * cs - p1 * sn, r1 = p1 * cs + p0 * sn;
-        x[i] = r0; x[i + half] = r1;
+        x[i0] = r0; x[i1] = r1;
         ss = fmaf(r0, r0, fmaf(r1, r1, ss));
     }
     for (int d = 2 * half + lane; d < a.D; d += 32) {
-        const float v = x[d] + (bias ? bias[d] : 0.f);
-        if (bias) x[d] = v;
+        float v = x[d] + (bias ? bias[d] : 0.f);
+        if (first) v *= inv * (w ? w[d] : 1.f);
+        if (bias || first) x[d] = v;
         ss = fmaf(v, v, ss);
     }
     __syncwarp();
-    float inv = 1.f;
-    if (a.norm) inv = 1.f / sqrtf(warp_sum(ss) / (float)a.D + a.eps);
-    const float* w = a.norm == 2 ? (is_k ? a.kw : a.qw) : nullptr;
+    if (first) { inv = 1.f; w = nullptr; }
+    else if (a.norm) inv = 1.f / sqrtf(warp_sum(ss) / (float)a.D + a.eps);
     if (is_k) {
         TC* dst = (TC*)a.kc + (((size_t)page * a.G + g) * a.PS + r) * a.D;
         for (int d = lane; d < a.D; d += 32) cstore<TC>(dst + d, x[d] * inv * (w ? w[d] : 1.f));
-    } else if (a.norm || a.q_mult) {
+    } else if ((a.norm && !first) || a.q_mult) {
         for (int d = lane; d < a.D; d += 32) x[d] = x[d] * inv * (w ? w[d] : 1.f) * qm;
     }
 }
@@ -213,6 +275,10 @@ struct AttnArgs {
     float scale, cap;
     int splits; float* ws;              // splits > 1: partial (m, l, acc[Dv]) records [row][H][splits][Dv + 2]
     unsigned* tickets;                  // one arrival counter per (tile, head block), zero between launches
+    int pool, pool_rows;                // pool > 0 (with a window): means of blocks of `pool` positions, rows per page of pk / pv
+    const void* pk; const void* pv;     // [pages][G][pool_rows][D] / [Dv], dense rows
+    const double* o_inv_freq;           // [Dv / 2] or NULL: pair m of an output (elements m and m + Dv / 2, or 2m and 2m + 1
+    int o_pairs;                        // with o_pairs) turns by -position * o_inv_freq[m]
 };
 
 constexpr int KT = 32;                  // keys per tile = one per lane
@@ -227,7 +293,33 @@ __device__ __forceinline__ int first_key(const AttnArgs& a, int pos) {
 }
 // The keys of a tile whose lowest window start is jlo come in two runs: the kept first positions below jlo, [0, kept), and
 // [jlo, jhi].  Key tile ti covers KT positions from tile_first(); positions past tile_last() are padding.
-__device__ __forceinline__ int kept_below(const AttnArgs& a, int jlo) { return a.window > 0 ? min(a.keep, jlo) : 0; }
+// With pooled blocks the first run is the blocks instead, [0, blocks_seen(last query)), a row of pk / pv each.
+__device__ __forceinline__ int blocks_seen(const AttnArgs& a, int pos) {
+    const int past = pos - a.window + 1;                 // positions below `past` have left the window
+    return past > 0 ? past / a.pool : 0;
+}
+__device__ __forceinline__ int early_rows(const AttnArgs& a, int jlo, int jhi) {
+    if (a.window <= 0) return 0;
+    return a.pool > 0 ? blocks_seen(a, jhi) : min(a.keep, jlo);
+}
+// element offset of pooled block b of KV head g, before the factor of the row size
+__device__ __forceinline__ long long pooled_row(const AttnArgs& a, int slot, int g, int b) {
+    const int e = b * a.pool + a.pool - 1, pg = e / a.PS;
+    const int page = a.table[(size_t)slot * a.max_pages + pg];
+    return ((long long)page * a.G + g) * a.pool_rows + (b - (int)((long long)pg * a.PS / a.pool));
+}
+// output element dv of a head turned back by the query's position, given its partner element (dv's pair)
+__device__ __forceinline__ int turn_partner(const AttnArgs& a, int dv) {
+    const int half = a.Dv >> 1;
+    return a.o_pairs ? dv ^ 1 : (dv < half ? dv + half : dv - half);
+}
+__device__ __forceinline__ float turn_back(const AttnArgs& a, int pos, int dv, float o, float partner) {
+    const int half = a.Dv >> 1;
+    const bool second = a.o_pairs ? (dv & 1) : dv >= half;
+    float sn, cs;
+    rope_angle_sincos(pos, a.o_inv_freq[a.o_pairs ? dv >> 1 : (second ? dv - half : dv)], sn, cs);
+    return second ? fmaf(o, cs, -partner * sn) : fmaf(o, cs, partner * sn);
+}
 __device__ __forceinline__ float distance_term(float slope, float slope2, bool log_form, int dist) {
     const float d = (float)max(dist, 0);
     return log_form ? slope * log1pf(slope2 * d) : slope * d;
@@ -323,17 +415,21 @@ __global__ void __launch_bounds__(256) seq_attention_kernel(AttnArgs a) {
     const TC* kc = (const TC*)a.kc;
     const TC* vc = (const TC*)a.vc;
     // this block's slice of the key tiles (all of them when splits == 1)
-    const int kept = kept_below(a, jlo), nkept = (kept + KT - 1) / KT;
+    const int kept = early_rows(a, jlo, jhi), nkept = (kept + KT - 1) / KT;
     const int ntile = nkept + (jhi - jlo) / KT + 1, per = (ntile + a.splits - 1) / a.splits;
     const int tbeg = (int)blockIdx.z * per, tend = min(ntile, tbeg + per);
     for (int ti = tbeg; ti < tend; ++ti) {
         const int j0 = ti < nkept ? ti * KT : jlo + (ti - nkept) * KT;
         const int jmax = ti < nkept ? kept - 1 : jhi;
+        const bool pooled = a.pool > 0 && ti < nkept;
         __syncthreads();
         if (threadIdx.x < KT) {
             const int j = j0 + threadIdx.x;
             long long ko = -1, vo = -1;
-            if (j <= jmax) {
+            if (pooled && j <= jmax) {
+                const long long pr = pooled_row(a, slot, g, j);
+                ko = pr * D; vo = pr * Dv;
+            } else if (j <= jmax) {
                 const int page = a.table[(size_t)slot * a.max_pages + j / a.PS], r = j % a.PS;
                 ko = (((long long)page * a.G + g) * a.PS + r) * a.kld;
                 vo = (((long long)page * a.G + g) * a.PS + r) * a.vld;
@@ -341,8 +437,8 @@ __global__ void __launch_bounds__(256) seq_attention_kernel(AttnArgs a) {
             krow[threadIdx.x] = ko; vrow[threadIdx.x] = vo;
         }
         __syncthreads();
-        stage_rows<TC>(Ks, DP, kc, krow, D, a.kld);
-        if (!a.valias) stage_rows<TC>(Vs, Dv, vc, vrow, Dv, a.vld);
+        stage_rows<TC>(Ks, DP, pooled ? (const TC*)a.pk : kc, krow, D, pooled ? D : a.kld);
+        if (!a.valias) stage_rows<TC>(Vs, Dv, pooled ? (const TC*)a.pv : vc, vrow, Dv, pooled ? Dv : a.vld);
         __syncthreads();
         if (!warp_live) continue;                   // a warp without a (query, head) pair only helps staging
         // scores: lane = key
@@ -362,7 +458,7 @@ __global__ void __launch_bounds__(256) seq_attention_kernel(AttnArgs a) {
             float sc = s[c] * a.scale;
             if (a.cap > 0.f) sc = a.cap * tanhf(sc / a.cap);
             sc -= distance_term(slope[c], slope2[c], log_form, pi[c] - j);
-            const bool vis = ok[c] && j <= jmax && j <= pi[c] && (j >= lo[c] || j < a.keep);
+            const bool vis = ok[c] && j <= jmax && (pooled ? j < blocks_seen(a, pi[c]) : (j <= pi[c] && (j >= lo[c] || j < a.keep)));
             if (a.prob) { p[c] = vis ? 1.f / (1.f + expf(-(sc + pb[c]))) : 0.f; continue; }
             sc = vis ? sc : -INFINITY;
             const float mn = fmaxf(m[c], warp_max(sc));
@@ -447,10 +543,33 @@ __global__ void __launch_bounds__(256) seq_attention_kernel(AttnArgs a) {
             float o = 0.f;
 #pragma unroll 8
             for (int sp = 0; sp < a.splits; ++sp) o = fmaf(wsl[p][sp], __ldcg(rec + (size_t)sp * (Dv + 2)), o);
+            if (a.o_inv_freq) {
+                const float* rp = rec - dv + turn_partner(a, dv);
+                float op = 0.f;
+#pragma unroll 8
+                for (int sp = 0; sp < a.splits; ++sp) op = fmaf(wsl[p][sp], __ldcg(rp + (size_t)sp * (Dv + 2)), op);
+                o = turn_back(a, pos0 + q, dv, o, op);
+            }
             if (a.gate) o *= 1.f / (1.f + expf(-gate_logit(a, t, h, dv)));
             a.out[t * a.ldo + (size_t)h * Dv + dv] = o * a.out_mult;
         }
         return;
+    }
+    if (a.o_inv_freq) {                                // a pair's elements meet through shared memory (the query tile is done)
+        float* ob = qs + warp * D * PPW;               // [D * PPW] floats of this warp; rows longer than that go through K's tile
+        const bool fits = Dv <= D * PPW;
+        if (!fits) { __syncthreads(); ob = Ks + warp * Dv; }
+#pragma unroll
+        for (int c = 0; c < PPW; ++c) {
+            __syncwarp();
+#pragma unroll
+            for (int v = 0; v < NV; ++v)
+                if (lane + 32 * v < Dv) ob[lane + 32 * v] = acc[c][v];
+            __syncwarp();
+#pragma unroll
+            for (int v = 0; v < NV; ++v)
+                if (ok[c] && lane + 32 * v < Dv) acc[c][v] = turn_back(a, pi[c], lane + 32 * v, acc[c][v], ob[turn_partner(a, lane + 32 * v)]);
+        }
     }
 #pragma unroll
     for (int c = 0; c < PPW; ++c) {
@@ -470,7 +589,11 @@ __global__ void __launch_bounds__(256) seq_attention_kernel(AttnArgs a) {
 
 template <typename TC, int NV>
 int launch_attn(const AttnArgs& a, int tiles, cudaStream_t st) {
-    const size_t smem = sizeof(float) * ((size_t)NWARP * a.D * PPW + (size_t)KT * (a.D + 1) + (a.valias ? 0 : (size_t)KT * a.Dv));
+    size_t smem = sizeof(float) * ((size_t)NWARP * a.D * PPW + (size_t)KT * (a.D + 1) + (a.valias ? 0 : (size_t)KT * a.Dv));
+    if (a.o_inv_freq) {                     // turning the outputs back needs a value row per warp behind the queries
+        const size_t turn = sizeof(float) * ((size_t)NWARP * a.D * PPW + (size_t)NWARP * a.Dv);
+        if (turn > smem) smem = turn;
+    }
     PGK_REQUIRE(smem <= 200 * 1024, "seq_attention failed: head sizes %d / %d need %zu bytes of shared memory", a.D, a.Dv, smem);
     static size_t configured = 0;
     // the opt-in is needed once dynamic + STATIC shared memory (row offsets, the fold's slice weights: ~9 KB) pass 48 KB
@@ -583,14 +706,16 @@ __global__ void __launch_bounds__(256) seq_attention_decode_kernel(AttnArgs a) {
     }
     // ... and the page of the warp's first key tile
     const int jlo = first_key(a, pos), jhi = pos;
-    const int kept = kept_below(a, jlo), nkept = (kept + KT - 1) / KT;
+    const int kept = early_rows(a, jlo, jhi), nkept = (kept + KT - 1) / KT;
     const int ntile = nkept + (jhi - jlo) / KT + 1, per = (ntile + a.splits - 1) / a.splits;
     const int tb = (int)blockIdx.z * per, te = min(ntile, tb + per);
     int page_first = 0;
     {
         const int ti = tb + warp;
-        const int j = (ti < nkept ? ti * KT : jlo + (ti - nkept) * KT) + lane;
-        if (ti < te && j <= (ti < nkept ? kept - 1 : jhi)) page_first = a.table[(size_t)slot * a.max_pages + j / a.PS];
+        const bool early = ti < nkept;
+        const int j = (early ? ti * KT : jlo + (ti - nkept) * KT) + lane;
+        const int at = a.pool > 0 && early ? j * a.pool + a.pool - 1 : j;          // a pooled block: its last position
+        if (ti < te && j <= (early ? kept - 1 : jhi)) page_first = a.table[(size_t)slot * a.max_pages + at / a.PS];
     }
     __syncthreads();
 
@@ -603,8 +728,6 @@ __global__ void __launch_bounds__(256) seq_attention_decode_kernel(AttnArgs a) {
 #pragma unroll
         for (int v = 0; v < NV; ++v) acc[p][v] = 0.f;
     }
-    const TC* kc = (const TC*)a.kc;
-    const TC* vc = (const TC*)a.vc;
     constexpr int KV = 16 / sizeof(TC);
     constexpr int VR = NV >= 16 ? 4 : 8;               // value rows in flight
     const bool kvec = D % KV == 0 && a.kld % KV == 0;
@@ -612,12 +735,21 @@ __global__ void __launch_bounds__(256) seq_attention_decode_kernel(AttnArgs a) {
     for (int ti = tb + warp; ti < te; ti += NWARP) {
         const int j0 = ti < nkept ? ti * KT : jlo + (ti - nkept) * KT, jmax = ti < nkept ? kept - 1 : jhi;
         const int j = j0 + lane;
-        const bool in = j <= jmax;
+        const bool in = j <= jmax, pooled = a.pool > 0 && ti < nkept;
+        const TC* kc = (const TC*)(pooled ? a.pk : a.kc);
+        const TC* vc = (const TC*)(pooled ? a.pv : a.vc);
         long long ko = 0, vo = 0;
         if (in) {
-            const int page = ti == tb + warp ? page_first : a.table[(size_t)slot * a.max_pages + j / a.PS], r = j % a.PS;
-            ko = (((long long)page * a.G + g) * a.PS + r) * a.kld;
-            vo = (((long long)page * a.G + g) * a.PS + r) * a.vld;
+            const int at = pooled ? j * a.pool + a.pool - 1 : j, pg = at / a.PS;
+            const int page = ti == tb + warp ? page_first : a.table[(size_t)slot * a.max_pages + pg];
+            const long long rk = (long long)page * a.G + g;
+            if (pooled) {
+                const long long pr = rk * a.pool_rows + (j - (int)((long long)pg * a.PS / a.pool));
+                ko = pr * D; vo = pr * Dv;
+            } else {
+                ko = (rk * a.PS + j % a.PS) * a.kld;
+                vo = (rk * a.PS + j % a.PS) * a.vld;
+            }
         }
         float s[DPAIRS];
 #pragma unroll
@@ -710,12 +842,13 @@ __global__ void __launch_bounds__(256) seq_attention_decode_kernel(AttnArgs a) {
     }
     __syncthreads();
     const size_t t = t0;
+    const bool turn = a.o_inv_freq && a.splits == 1;
     for (int i = threadIdx.x; i < nh * Dv; i += blockDim.x) {
-        const int p = i / Dv, dv = i - p * Dv;
+        const int p = i / Dv, dv = i - p * Dv, dp = turn ? turn_partner(a, dv) : dv;
         float M = -INFINITY;
 #pragma unroll
         for (int w = 0; w < NWARP; ++w) M = fmaxf(M, st_m[w * DPAIRS + p]);
-        float L = 0.f, o = 0.f;
+        float L = 0.f, o = 0.f, op = 0.f;
 #pragma unroll
         for (int w = 0; w < NWARP; ++w) {
             const float mw = st_m[w * DPAIRS + p];
@@ -723,8 +856,10 @@ __global__ void __launch_bounds__(256) seq_attention_decode_kernel(AttnArgs a) {
                 const float e = expf(mw - M);
                 L = fmaf(st_l[w * DPAIRS + p], e, L);
                 o = fmaf(st_acc[((size_t)w * DPAIRS + p) * Dv + dv], e, o);
+                if (turn) op = fmaf(st_acc[((size_t)w * DPAIRS + p) * Dv + dp], e, op);
             }
         }
+        if (turn) o = turn_back(a, pos, dv, o, op);
         const int h = hb0 + p;
         if (a.splits > 1) {
             float* rec = a.ws + ((t * a.H + h) * a.splits + blockIdx.z) * (Dv + 2);
@@ -785,6 +920,13 @@ __global__ void __launch_bounds__(256) seq_attention_decode_kernel(AttnArgs a) {
         float o = 0.f;
 #pragma unroll 8
         for (int sp = 0; sp < a.splits; ++sp) o = fmaf(wsl[p][sp], __ldcg(rec + (size_t)sp * (Dv + 2)), o);
+        if (a.o_inv_freq) {
+            const float* rp = rec - dv + turn_partner(a, dv);
+            float op = 0.f;
+#pragma unroll 8
+            for (int sp = 0; sp < a.splits; ++sp) op = fmaf(wsl[p][sp], __ldcg(rp + (size_t)sp * (Dv + 2)), op);
+            o = turn_back(a, pos, dv, o, op);
+        }
         if (a.gate) {
             const int u = (i - (int)threadIdx.x) >> 8;
             float z = 0.f;
@@ -879,6 +1021,24 @@ int pgk_seq_attention_ex2(const float* q, int ldq, int q_off, const float* gate_
                           int vdim, int chunk, int window, int keep_first, float scale, float softcap, int weight_mode,
                           const float* weight_bias, float out_mult, int splits, float* workspace, uint32_t* tickets,
                           int single_query, void* stream) {
+    return pgk_seq_attention_ex3(q, ldq, q_off, gate_rows, ldg, gate_off, gate_mode, out, ldo, k_cache, v_cache, k_ld, v_ld,
+                                 cache_dtype, table, max_pages, page_size, tiles, n_tiles, slopes, slopes2, sinks, heads, kv_heads,
+                                 dim, vdim, chunk, window, keep_first, scale, softcap, weight_mode, weight_bias, out_mult, 0, 0,
+                                 nullptr, nullptr, nullptr, 0, splits, workspace, tickets, single_query, stream);
+}
+
+int pgk_seq_attention_ex3(const float* q, int ldq, int q_off, const float* gate_rows, int ldg, int gate_off, int gate_mode,
+                          float* out, int ldo, const void* k_cache, const void* v_cache, int k_ld, int v_ld, int cache_dtype,
+                          const int32_t* table, int max_pages, int page_size, const int32_t* tiles, int n_tiles,
+                          const float* slopes, const float* slopes2, const float* sinks, int heads, int kv_heads, int dim,
+                          int vdim, int chunk, int window, int keep_first, float scale, float softcap, int weight_mode,
+                          const float* weight_bias, float out_mult, int pool, int pool_rows, const void* k_pool,
+                          const void* v_pool, const double* out_inv_freq, int out_pairs, int splits, float* workspace,
+                          uint32_t* tickets, int single_query, void* stream) {
+    PGK_REQUIRE(pool >= 0 && (pool == 0 || (window > 0 && chunk == 0 && keep_first == 0 && !slopes && k_pool && v_pool &&
+                                            pool_rows >= (page_size + pool - 1) / pool)),
+                "seq_attention failed: pooled blocks need a window, their two arrays with enough rows per page, no chunks, no kept positions and no distance term");
+    PGK_REQUIRE(!out_inv_freq || vdim % 2 == 0, "seq_attention failed: outputs of an odd size %d cannot turn in pairs", vdim);
     PGK_REQUIRE(keep_first >= 0 && (keep_first == 0 || (window > 0 && chunk == 0)),
                 "seq_attention failed: kept first positions need a window and no chunks");
     PGK_REQUIRE(!slopes2 || slopes, "seq_attention failed: the logarithmic distance term needs both per-head vectors");
@@ -901,6 +1061,8 @@ int pgk_seq_attention_ex2(const float* q, int ldq, int q_off, const float* gate_
     a.H = heads; a.G = kv_heads; a.D = dim; a.Dv = vdim; a.chunk = chunk;
     a.HB = pgk_seq_heads_per_block(heads, kv_heads); a.gate = gate_mode;
     a.scale = scale; a.cap = softcap; a.splits = splits; a.ws = workspace; a.tickets = tickets;
+    a.pool = pool; a.pool_rows = pool_rows; a.pk = k_pool; a.pv = v_pool; a.o_inv_freq = out_inv_freq; a.o_pairs = out_pairs;
+    PGK_REQUIRE(!a.valias || pool == 0, "seq_attention failed: pooled blocks keep their values in an array of their own");
     if (single_query)       // every tile holds one query: the decoding kernel
         return cache_dtype == 2 ? launch_attn_decode_nv<uint16_t>(a, n_tiles, (cudaStream_t)stream)
                                 : launch_attn_decode_nv<float>(a, n_tiles, (cudaStream_t)stream);
@@ -950,6 +1112,22 @@ int pgk_seq_mixer_prep_rot_ex(float* proj, int ld, int tokens, int heads, int kv
                               const float* k_weight, float eps, const float* q_bias, const float* k_bias, const float* v_bias,
                               const float* q_mult, void* k_cache, void* v_cache, int cache_dtype, const int32_t* table,
                               int max_pages, int page_size, const int32_t* slot, const int32_t* pos, void* stream) {
+    return pgk_seq_mixer_prep_rot_ex2(proj, ld, tokens, heads, kv_heads, dim, vdim, q_off, k_off, v_off, rot_dims, inv_freq, norm_mode,
+                                      q_weight, k_weight, eps, q_bias, k_bias, v_bias, q_mult, 0, 0, nullptr, 0, 0, nullptr, nullptr, 0,
+                                      k_cache, v_cache, cache_dtype, table, max_pages, page_size, slot, pos, stream);
+}
+
+// ---- the same with the pair layout, the norm in front of the rotation, rotated values and pooled blocks
+int pgk_seq_mixer_prep_rot_ex2(float* proj, int ld, int tokens, int heads, int kv_heads, int dim, int vdim, int q_off, int k_off,
+                               int v_off, int rot_dims, const double* inv_freq, int norm_mode, const float* q_weight,
+                               const float* k_weight, float eps, const float* q_bias, const float* k_bias, const float* v_bias,
+                               const float* q_mult, int pairs, int norm_first, const double* v_inv_freq, int pool, int pool_rows,
+                               void* k_pool, void* v_pool, int single_token, void* k_cache, void* v_cache, int cache_dtype,
+                               const int32_t* table, int max_pages, int page_size, const int32_t* slot, const int32_t* pos,
+                               void* stream) {
+    PGK_REQUIRE(!v_inv_freq || vdim % 2 == 0, "seq_mixer_prep_rot failed: values of an odd size %d cannot turn in pairs", vdim);
+    PGK_REQUIRE(pool >= 0 && (pool == 0 || (k_pool && v_pool && pool_rows >= (page_size + pool - 1) / pool)),
+                "seq_mixer_prep_rot failed: pooled blocks of %d positions need both arrays with enough rows per page", pool);
     PGK_REQUIRE(cache_dtype == 0 || cache_dtype == 2, "seq_mixer_prep_rot failed: the cache is float32 (0) or bfloat16 (2), got %d", cache_dtype);
     PGK_REQUIRE(heads > 0 && kv_heads > 0 && heads % kv_heads == 0 && dim > 0 && vdim > 0, "seq_mixer_prep_rot failed: invalid head layout");
     PGK_REQUIRE(rot_dims >= 0 && rot_dims % 2 == 0 && rot_dims <= dim && (rot_dims == 0 || inv_freq),
@@ -957,10 +1135,17 @@ int pgk_seq_mixer_prep_rot_ex(float* proj, int ld, int tokens, int heads, int kv
     PGK_REQUIRE(norm_mode >= 0 && norm_mode <= 2 && (norm_mode != 2 || (q_weight && k_weight)), "seq_mixer_prep_rot failed: norm mode %d", norm_mode);
     if (tokens <= 0) return 0;
     PrepRotArgs a{proj, ld, heads, kv_heads, dim, vdim, q_off, k_off, v_off, rot_dims, inv_freq, norm_mode, q_weight, k_weight, eps,
-                  k_cache, v_cache, table, max_pages, page_size, slot, pos, q_bias, k_bias, v_bias, q_mult};
-    const dim3 grid(tokens, (heads + 2 * kv_heads + 3) / 4);
+                  k_cache, v_cache, table, max_pages, page_size, slot, pos, q_bias, k_bias, v_bias, q_mult, pairs ? 1 : 0,
+                  norm_first ? 1 : 0, v_inv_freq, single_token ? pool : 0, pool_rows, k_pool, v_pool};
+    const dim3 grid(tokens, (heads + (a.pool > 0 ? 4 : 2) * kv_heads + 3) / 4);
     if (cache_dtype == 2) PGK_CUDA(launch(mixer_prep_rot_kernel<uint16_t>, grid, dim3(128), 0, (cudaStream_t)stream, a));
     else PGK_CUDA(launch(mixer_prep_rot_kernel<float>, grid, dim3(128), 0, (cudaStream_t)stream, a));
+    if (pool > 0 && !single_token) {        // rows of the same step may complete a block: pooled behind the launch that writes them
+        a.pool = pool;
+        const dim3 pg(tokens, (2 * kv_heads + 3) / 4);
+        if (cache_dtype == 2) PGK_CUDA(launch(pool_rows_kernel<uint16_t>, pg, dim3(128), 0, (cudaStream_t)stream, a));
+        else PGK_CUDA(launch(pool_rows_kernel<float>, pg, dim3(128), 0, (cudaStream_t)stream, a));
+    }
     return 0;
 }
 

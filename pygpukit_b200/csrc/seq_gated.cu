@@ -7,6 +7,7 @@
 //   moe_route_biased   softmax over all router outputs; the `top` largest of score + bias are chosen, their weights are the
 //                      scores themselves (renormalised on request); router outputs >= real_experts stand for experts without
 //                      matrices (`mat` = -1 for them)
+//   moe_route_logits   a bias on the logits, the `top` largest logits chosen, weights = softmax over the chosen ones only
 //   moe_combine_rows   out = sum_k w[t, k] * (parts row, or the token's own input row for an expert without matrices)
 //                      + sigmoid(gate logit) * shared expert row
 //   dyt_seam           a sublayer's result (plain rows, the two-branch join, or the expert sum) through the norm behind it into
@@ -147,6 +148,52 @@ __global__ void __launch_bounds__(ROUTE_WARPS * 32) moe_route_biased_kernel(Rout
     if (a.renorm) {
         __syncwarp();
         for (int k = lane; k < a.top; k += 32) a.wt[(size_t)t * a.top + k] /= (wsum + 1e-20f);
+    }
+}
+
+// ---------------------------------------------------------------- router that chooses and weighs by the logits
+// One warp per token: z + bias, the `top` largest in order, then a softmax over those alone.  With `extra` >= 0 every token also
+// takes that matrix with weight 1 as its last slot (a shared expert that rides in the experts' stack).
+struct RouteLogitsArgs {
+    const float* z; int ldz, T, E, top, extra;
+    const float* bias;
+    int* idx; float* wt; int* rank; int* counts;
+};
+
+__global__ void __launch_bounds__(ROUTE_WARPS * 32) moe_route_logits_kernel(RouteLogitsArgs a) {
+    extern __shared__ float sm[];
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    const int t = blockIdx.x * ROUTE_WARPS + warp;
+    if (t >= a.T) return;
+    float* c = sm + (size_t)warp * a.E;
+    const float* z = a.z + (size_t)t * a.ldz;
+    for (int e = lane; e < a.E; e += 32) c[e] = z[e] + (a.bias ? a.bias[e] : 0.f);
+    __syncwarp();
+    const int slots = a.top + (a.extra >= 0 ? 1 : 0);
+    const size_t o = (size_t)t * slots;
+    float zmax = 0.f, sum = 0.f;
+    for (int k = 0; k < a.top; ++k) {
+        float bv = -INFINITY; int bi = 0x7fffffff;
+        for (int e = lane; e < a.E; e += 32)
+            if (c[e] > bv || bi == 0x7fffffff) { bv = c[e]; bi = e; }
+        warp_argmax(bv, bi);
+        if (k == 0) zmax = bv;
+        const float p = expf(bv - zmax);
+        sum += p;
+        __syncwarp();
+        if (lane == 0) {
+            c[bi] = -INFINITY;
+            a.idx[o + k] = bi;
+            a.wt[o + k] = p;
+            if (a.counts) a.rank[o + k] = atomicAdd(&a.counts[bi], 1);
+        }
+        __syncwarp();
+    }
+    for (int k = lane; k < a.top; k += 32) a.wt[o + k] /= sum;
+    if (a.extra >= 0 && lane == 0) {
+        a.idx[o + a.top] = a.extra;
+        a.wt[o + a.top] = 1.f;
+        if (a.counts) a.rank[o + a.top] = atomicAdd(&a.counts[a.extra], 1);
     }
 }
 
@@ -312,15 +359,6 @@ struct GatedArgs {
     int H, G, D, Dv;
     int vec;                          // every row, offset and size a multiple of 16 bytes: chunks arrive by asynchronous copies
 };
-
-__device__ __forceinline__ void cp_async16(void* smem, const void* g) {
-    asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_u32(smem)), "l"(g) : "memory");
-}
-__device__ __forceinline__ void cp_async4(void* smem, const void* g) {
-    asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"(smem_u32(smem)), "l"(g) : "memory");
-}
-__device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
-template <int N> __device__ __forceinline__ void cp_async_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
 
 // One stage of the chunk pipeline in shared memory: Q [GTC][Dp], K [GTC][Dp], then the decays [GTC][Dp] (gated outer product)
 // or g, beta and q.k per token [3][GTC] (delta rule), then V [GTC][GCOLS].  Dp = D rounded up to 4 GR; rows D .. Dp - 1 and value
@@ -580,6 +618,19 @@ int pgk_moe_route_biased(const float* logits, int ld, int tokens, int outputs, i
     const size_t smem = (size_t)ROUTE_WARPS * 2 * outputs * 4;
     PGK_REQUIRE(smem <= 48 * 1024, "moe_route_biased failed: too many router outputs (%d)", outputs);
     PGK_CUDA(launch(moe_route_biased_kernel, dim3((tokens + ROUTE_WARPS - 1) / ROUTE_WARPS), dim3(ROUTE_WARPS * 32), smem,
+                    (cudaStream_t)stream, a));
+    return 0;
+}
+
+int pgk_moe_route_logits(const float* logits, int ld, int tokens, int experts, int top, const float* bias, int extra, int32_t* idx,
+                         float* weights, int32_t* rank, int32_t* counts, void* stream) {
+    PGK_REQUIRE(experts > 0 && top > 0 && top <= experts, "moe_route_logits failed: top %d of %d experts", top, experts);
+    PGK_REQUIRE((rank == nullptr) == (counts == nullptr), "moe_route_logits failed: ranks and counts come together");
+    if (tokens <= 0) return 0;
+    RouteLogitsArgs a{logits, ld, tokens, experts, top, extra, bias, idx, weights, rank, counts};
+    const size_t smem = (size_t)ROUTE_WARPS * experts * 4;
+    PGK_REQUIRE(smem <= 48 * 1024, "moe_route_logits failed: too many experts (%d)", experts);
+    PGK_CUDA(launch(moe_route_logits_kernel, dim3((tokens + ROUTE_WARPS - 1) / ROUTE_WARPS), dim3(ROUTE_WARPS * 32), smem,
                     (cudaStream_t)stream, a));
     return 0;
 }

@@ -11,7 +11,8 @@
 //   * epilogues: plain; gate/up pairs (W holds gate_j in row 2j and up_j in row 2j + 1, the output is silu(gate) * up,
 //     [M, N / 2]); scale then tanh cap (the logit head); clamped gate/up pairs g = min(gate, limit), u = clamp(up, +-limit),
 //     output g sigmoid(alpha g) (u + 1); C += column vector * product (layer scale and residual add in one pass);
-//     gelu_tanh(product) * gathered table entry (per-layer token inputs);
+//     gelu_tanh(product) * gathered table entry (per-layer token inputs); squared ReLU; gate/up pairs with gelu_tanh(gate) * up;
+//     gelu_erf(product);
 //   * batches: grid.z can also walk `batch` independent products whose A columns, matrices and C columns are a fixed number
 //     of elements apart (one product per attention head on slices of the same rows).
 #include "common.cuh"
@@ -41,6 +42,7 @@ struct GemmArgs {
 __device__ __forceinline__ float gelu_tanh_f(float z) {
     return 0.5f * z * (1.f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
 }
+__device__ __forceinline__ float gelu_erf_f(float z) { return 0.5f * z * (1.f + erff(z * 0.7071067811865476f)); }
 __device__ __forceinline__ float aux_at(const GemmArgs& a, int row, int col) {
     const size_t i = (size_t)a.aux_rows[row] * a.aux_ld + a.aux_off + col;
     return a.aux_dt == 2 ? bf16_bits_to_f32(((const uint16_t*)a.aux)[i]) : ((const float*)a.aux)[i];
@@ -53,6 +55,10 @@ __device__ __forceinline__ void store_pair(const GemmArgs& a, int row, int col, 
     // (row, col) and (row, col + 1), col even
     if (EPI == 1) {
         if (col + 1 < a.N) a.C[(size_t)row * a.ldc + (col >> 1)] = silu_f(c0) * c1;
+        return;
+    }
+    if (EPI == 7) {
+        if (col + 1 < a.N) a.C[(size_t)row * a.ldc + (col >> 1)] = gelu_tanh_f(c0) * c1;
         return;
     }
     if (EPI == 3) {          // scale = alpha, cap = limit
@@ -70,6 +76,7 @@ __device__ __forceinline__ void store_pair(const GemmArgs& a, int row, int col, 
         c0 = fmaxf(c0, 0.f); c1 = fmaxf(c1, 0.f);
         c0 *= c0; c1 *= c1;
     }
+    if (EPI == 8) { c0 = gelu_erf_f(c0); c1 = gelu_erf_f(c1); }
     float* p = a.C + (size_t)row * a.ldc + col;
     if (EPI == 4) {
         if (col < a.N) p[0] = fmaf(a.colv[col], c0, p[0]);
@@ -479,8 +486,8 @@ int pgk_gemm_rows_f32(const float* A, int lda, const int32_t* a_rows, const void
                       int epilogue, float scale, float cap, void* stream) {
     PGK_REQUIRE(wdt == 0 || wdt == 2, "gemm_rows_f32 failed: weights must be float32 (0) or bfloat16 (2), got %d", wdt);
     PGK_REQUIRE(N > 0 && K > 0 && M >= 0, "gemm_rows_f32 failed: invalid shape M=%d N=%d K=%d", M, N, K);
-    PGK_REQUIRE(epilogue >= 0 && epilogue <= 2, "gemm_rows_f32 failed: unknown epilogue %d", epilogue);
-    PGK_REQUIRE(epilogue != 1 || N % 2 == 0, "gemm_rows_f32 failed: the gate/up epilogue needs an even N");
+    PGK_REQUIRE((epilogue >= 0 && epilogue <= 2) || epilogue == 7 || epilogue == 8, "gemm_rows_f32 failed: unknown epilogue %d", epilogue);
+    PGK_REQUIRE((epilogue != 1 && epilogue != 7) || N % 2 == 0, "gemm_rows_f32 failed: the gate/up epilogue needs an even N");
     const int G = group_off ? groups : 1;
     const int rows = group_off ? max_rows : M;
     if (rows <= 0 || G <= 0) return 0;
@@ -492,6 +499,8 @@ int pgk_gemm_rows_f32(const float* A, int lda, const int32_t* a_rows, const void
     }
     if (epilogue == 0) return launch_many<0>(a, wdt, G, rows, st);
     if (epilogue == 1) return launch_many<1>(a, wdt, G, rows, st);
+    if (epilogue == 7) return launch_many<7>(a, wdt, G, rows, st);
+    if (epilogue == 8) return launch_many<8>(a, wdt, G, rows, st);
     return launch_many<2>(a, wdt, G, rows, st);
 }
 
@@ -504,13 +513,15 @@ int pgk_gemm_few_rows_f32(const float* A, int lda, const int32_t* a_rows, const 
     PGK_REQUIRE(N > 0 && K > 0 && M >= 0, "gemm_few_rows_f32 failed: invalid shape M=%d N=%d K=%d", M, N, K);
     PGK_REQUIRE(rows_per_block >= 1 && rows_per_block <= RMAX, "gemm_few_rows_f32 failed: 1..%d rows per block", RMAX);
     PGK_REQUIRE((size_t)rows_per_block * K * 4 <= 200 * 1024, "gemm_few_rows_f32 failed: %d rows of K=%d do not fit shared memory", rows_per_block, K);
-    PGK_REQUIRE(epilogue >= 0 && epilogue <= 2, "gemm_few_rows_f32 failed: unknown epilogue %d", epilogue);
-    PGK_REQUIRE(epilogue != 1 || N % 2 == 0, "gemm_few_rows_f32 failed: the gate/up epilogue needs an even N");
+    PGK_REQUIRE((epilogue >= 0 && epilogue <= 2) || epilogue == 7 || epilogue == 8, "gemm_few_rows_f32 failed: unknown epilogue %d", epilogue);
+    PGK_REQUIRE((epilogue != 1 && epilogue != 7) || N % 2 == 0, "gemm_few_rows_f32 failed: the gate/up epilogue needs an even N");
     if (M == 0) return 0;
     GemmArgs a{A, a_rows, W, C, nullptr, row_group, w_group_stride, lda, ldc, M, N, K, scale, cap, nullptr, nullptr, nullptr, 0, 0, 0, 0, 0};
     cudaStream_t st = (cudaStream_t)stream;
     if (epilogue == 0) return launch_few<0>(a, wdt, rows_per_block, st);
     if (epilogue == 1) return launch_few<1>(a, wdt, rows_per_block, st);
+    if (epilogue == 7) return launch_few<7>(a, wdt, rows_per_block, st);
+    if (epilogue == 8) return launch_few<8>(a, wdt, rows_per_block, st);
     return launch_few<2>(a, wdt, rows_per_block, st);
 }
 
@@ -524,8 +535,8 @@ int pgk_gemm_seq_f32(const float* A, int lda, long long a_batch, const void* W, 
                      void* stream) {
     PGK_REQUIRE(wdt == 0 || wdt == 2, "gemm_seq_f32 failed: weights must be float32 (0) or bfloat16 (2), got %d", wdt);
     PGK_REQUIRE(N > 0 && K > 0 && M >= 0 && batch >= 1, "gemm_seq_f32 failed: invalid shape M=%d N=%d K=%d batch=%d", M, N, K, batch);
-    PGK_REQUIRE(epilogue >= 0 && epilogue <= 6, "gemm_seq_f32 failed: unknown epilogue %d", epilogue);
-    PGK_REQUIRE((epilogue != 1 && epilogue != 3) || N % 2 == 0, "gemm_seq_f32 failed: a gate/up epilogue needs an even N");
+    PGK_REQUIRE(epilogue >= 0 && epilogue <= 8, "gemm_seq_f32 failed: unknown epilogue %d", epilogue);
+    PGK_REQUIRE((epilogue != 1 && epilogue != 3 && epilogue != 7) || N % 2 == 0, "gemm_seq_f32 failed: a gate/up epilogue needs an even N");
     PGK_REQUIRE(epilogue != 4 || col_scale, "gemm_seq_f32 failed: the scaled-accumulate epilogue needs its column factors");
     PGK_REQUIRE(epilogue != 5 || (aux && aux_rows && (aux_dtype == 0 || aux_dtype == 2)), "gemm_seq_f32 failed: the gather epilogue needs its table and rows");
     PGK_REQUIRE(rows_per_block >= 0 && rows_per_block <= RMAX, "gemm_seq_f32 failed: 0..%d rows per block", RMAX);
@@ -541,7 +552,9 @@ int pgk_gemm_seq_f32(const float* A, int lda, long long a_batch, const void* W, 
             case 3: return launch_few<3>(a, wdt, rows_per_block, st, batch);
             case 4: return launch_few<4>(a, wdt, rows_per_block, st, batch);
             case 5: return launch_few<5>(a, wdt, rows_per_block, st, batch);
-            default: return launch_few<6>(a, wdt, rows_per_block, st, batch);
+            case 6: return launch_few<6>(a, wdt, rows_per_block, st, batch);
+            case 7: return launch_few<7>(a, wdt, rows_per_block, st, batch);
+            default: return launch_few<8>(a, wdt, rows_per_block, st, batch);
         }
     }
     switch (epilogue) {
@@ -551,7 +564,9 @@ int pgk_gemm_seq_f32(const float* A, int lda, long long a_batch, const void* W, 
         case 3: return launch_many<3>(a, wdt, batch, M, st);
         case 4: return launch_many<4>(a, wdt, batch, M, st);
         case 5: return launch_many<5>(a, wdt, batch, M, st);
-        default: return launch_many<6>(a, wdt, batch, M, st);
+        case 6: return launch_many<6>(a, wdt, batch, M, st);
+        case 7: return launch_many<7>(a, wdt, batch, M, st);
+        default: return launch_many<8>(a, wdt, batch, M, st);
     }
 }
 

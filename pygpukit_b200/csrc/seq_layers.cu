@@ -153,6 +153,90 @@ __global__ void __launch_bounds__(256) rms_seam_kernel(RmsSeamArgs a) {
     for (int i = threadIdx.x; i < a.W; i += blockDim.x) a.h[o + i] = row[i] * inv2 * (a.off2 + a.w2[i]);
 }
 
+// y = base[t] (may be absent) + sum_k w[t, k] * parts[inv[t, k]];  x[t] += rms(y) * weight: a sublayer's result -- plain rows, or
+// the weighted expert rows with the shared expert's -- joins the residual stream behind its RMS norm in one launch.  A thread
+// keeps its share of the row in registers (up to 16 elements: four 16-byte groups, or 16 strided ones when the rows are not
+// 16-byte aligned); the block has as many threads as the row needs.
+struct RmsJoinArgs {
+    const float* base; const float* parts; const int* inv; const float* w; int top;
+    const float* weight; float eps;
+    float* x; int W;
+};
+
+constexpr int JOIN_MAX = 16;         // elements per thread
+
+template <bool VEC>
+__global__ void __launch_bounds__(1024) rms_join_kernel(RmsJoinArgs a) {
+    __shared__ float red[32];
+    __shared__ float wk[TOPMAX];
+    __shared__ long long pk[TOPMAX];
+    constexpr int E = VEC ? 4 : 1;
+    const int t = blockIdx.x, tid = threadIdx.x, nt = blockDim.x, top = a.top;
+    const size_t o = (size_t)t * a.W;
+    float v[JOIN_MAX], xv[JOIN_MAX];
+#pragma unroll
+    for (int j = 0; j < JOIN_MAX / E; ++j) {          // what depends on nothing but the row goes out first
+        const int i = (tid + j * nt) * E;
+        if (i >= a.W) continue;
+        if (VEC) {
+            *(float4*)&xv[j * E] = *(const float4*)(a.x + o + i);
+            *(float4*)&v[j * E] = a.base ? *(const float4*)(a.base + o + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+        } else {
+            xv[j] = a.x[o + i];
+            v[j] = a.base ? a.base[o + i] : 0.f;
+        }
+    }
+    if (top > 0) {
+        for (int k0 = 0; k0 < top; k0 += TOPMAX) {
+            const int kn = min(TOPMAX, top - k0);
+            __syncthreads();
+            if (tid < kn) {
+                wk[tid] = a.w[(size_t)t * top + k0 + tid];
+                pk[tid] = (long long)a.inv[(size_t)t * top + k0 + tid] * a.W;
+            }
+            __syncthreads();
+#pragma unroll
+            for (int j = 0; j < JOIN_MAX / E; ++j) {
+                const int i = (tid + j * nt) * E;
+                if (i >= a.W) continue;
+#pragma unroll 4
+                for (int k = 0; k < kn; ++k) {
+                    if (VEC) {
+                        const float4 p = *(const float4*)(a.parts + pk[k] + i);
+                        const float pp[4] = {p.x, p.y, p.z, p.w};
+#pragma unroll
+                        for (int e = 0; e < E; ++e) v[j * E + e] = fmaf(wk[k], pp[e], v[j * E + e]);
+                    } else {
+                        v[j] = fmaf(wk[k], a.parts[pk[k] + i], v[j]);
+                    }
+                }
+            }
+        }
+    }
+    float q = 0.f;
+#pragma unroll
+    for (int j = 0; j < JOIN_MAX / E; ++j) {
+        if ((tid + j * nt) * E >= a.W) continue;
+#pragma unroll
+        for (int e = 0; e < E; ++e) q = fmaf(v[j * E + e], v[j * E + e], q);
+    }
+    q = warp_sum(q);
+    if ((tid & 31) == 0) red[tid >> 5] = q;
+    __syncthreads();
+    float s = 0.f;
+    for (int i = 0; i < (nt >> 5); ++i) s += red[i];
+    const float inv = 1.f / sqrtf(s / (float)a.W + a.eps);
+#pragma unroll
+    for (int j = 0; j < JOIN_MAX / E; ++j) {
+        const int i = (tid + j * nt) * E;
+        if (i >= a.W) continue;
+#pragma unroll
+        for (int e = 0; e < E; ++e) xv[j * E + e] += v[j * E + e] * inv * a.weight[i + e];
+        if (VEC) *(float4*)(a.x + o + i) = *(const float4*)&xv[j * E];
+        else a.x[o + i] = xv[j];
+    }
+}
+
 // x[t] = rms(table[tokens[t]]) * (off + w), copied to keep[t] as well when given: embedding, its norm and the kept copy
 template <typename TW>
 __global__ void __launch_bounds__(256) embed_norm_rows_kernel(const TW* table, const int* tok, const float* w, float off, float eps,
@@ -333,6 +417,23 @@ int pgk_rms_norm_seam_f32(const float* y, const float* weight1, float offset1, f
         configured = true;
     }
     PGK_CUDA(launch(rms_seam_kernel, dim3(rows), dim3(256), smem, (cudaStream_t)stream, a));
+    return 0;
+}
+
+int pgk_rms_join_f32(const float* base, const float* parts, const int32_t* inv, const float* weights, int top, const float* weight,
+                     float eps, float* x, int rows, int width, void* stream) {
+    PGK_REQUIRE(width > 0 && width <= 1024 * JOIN_MAX, "rms_join_f32 failed: width %d out of range", width);
+    PGK_REQUIRE(top >= 0 && (base || top > 0) && (top == 0 || (parts && inv && weights)), "rms_join_f32 failed: parts need their index and weights");
+    if (rows <= 0) return 0;
+    RmsJoinArgs a{base, parts, inv, weights, top, weight, eps, x, width};
+    const bool vec = width % 4 == 0 && (((uintptr_t)base | (uintptr_t)parts | (uintptr_t)x | (uintptr_t)weight) & 15) == 0;
+    const int units = vec ? width / 4 : width;
+    int nt = rows <= 32 ? (units + 31) / 32 * 32 : (units + 63) / 64 * 32;      // few rows: one group per thread
+    if (nt < 64) nt = 64;
+    if (nt > 1024) nt = 1024;
+    while ((long long)nt * JOIN_MAX < width && nt < 1024) nt += 32;
+    if (vec) PGK_CUDA(launch(rms_join_kernel<true>, dim3(rows), dim3(nt), 0, (cudaStream_t)stream, a));
+    else PGK_CUDA(launch(rms_join_kernel<false>, dim3(rows), dim3(nt), 0, (cudaStream_t)stream, a));
     return 0;
 }
 

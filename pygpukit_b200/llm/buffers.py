@@ -107,7 +107,7 @@ class RowBuffers:
             if L.mlp is not None and L.mlp.kind == "dense":
                 sff = max(sff, L.mlp.ff)
             elif L.mlp is not None:
-                top, ff, sff = max(top, L.mlp.top), max(ff, L.mlp.ff), max(sff, L.mlp.shared_ff)
+                top, ff, sff = max(top, getattr(L.mlp, "slots", L.mlp.top)), max(ff, L.mlp.ff), max(sff, L.mlp.shared_ff)
                 experts = max(experts, getattr(L.mlp, "routes", L.mlp.experts) + 1)
         R = self.rows = max(8, int(rows))
         self.x = GPUArray((R, W), float32)

@@ -249,7 +249,12 @@ class AttentionMixerSpec:
     `norm_weight` False divides q and k by their root mean square and multiplies by nothing.  `weights` "softmax", or
     "sigmoid": the weight of a visible key is sigmoid(score + b_h) with a learned number per head, not normalised.
     `qkv_bias`: the q, k and v projections have biases (added before the rotation).  `head_temp`: the score is also
-    multiplied by a learned number per head."""
+    multiplied by a learned number per head.
+
+    `norm_first`: the q / k norm comes before the rotation instead of behind it.  `rot_values`: the values are rotated by their
+    position too (over all vdim elements, the rotation's base and layout) and cached so; every head's output is turned back by
+    the query's position.  `pool` > 0 (with a window): beside its window a query at i sees one key and one value for every block
+    of `pool` positions that ends at or before i - window, the means of the cached ones, in the same softmax."""
     heads: int
     kv_heads: int
     dim: int
@@ -273,6 +278,9 @@ class AttentionMixerSpec:
     weights: str = "softmax"
     qkv_bias: bool = False
     head_temp: bool = False
+    norm_first: bool = False
+    rot_values: bool = False
+    pool: int = 0
 
     kind = "attention"
 
@@ -304,14 +312,20 @@ class AttentionMixerSpec:
 
 @dataclass(frozen=True)
 class RotarySpec:
-    """Rotary positions in the half layout: of the first `dims` elements of a head, element i is paired with element
-    i + dims / 2 and the pair turns by position * base^(-2 i / dims) / factor (`factor`: linear position scaling)."""
+    """Rotary positions on the first `dims` elements of a head: pair i turns by position * base^(-2 i / dims) / factor
+    (`factor`: linear position scaling).  `layout` "half": element i is paired with element i + dims / 2; "pairs": element 2i
+    with element 2i + 1."""
     dims: int
     base: float
     factor: float = 1.0
+    layout: str = "half"
 
     def inv_freq(self) -> list[float]:
         return [self.base ** (-2.0 * i / self.dims) / self.factor for i in range(self.dims // 2)]
+
+    def value_inv_freq(self, vdim: int) -> list[float]:
+        """the same base over all `vdim` elements of a value, without position scaling"""
+        return [self.base ** (-2.0 * i / vdim) for i in range(vdim // 2)]
 
 
 @dataclass(frozen=True)
@@ -431,6 +445,43 @@ class DeltaMixerSpec:
 
 
 @dataclass(frozen=True)
+class MatrixLSTMSpec:
+    """The matrix memory of xLSTM with a float32 state per sequence: per head S_t = e^f S_(t-1) + e^i k v^T and n_t likewise
+    with k alone, kept in range by a running maximum m of the log gates (m = 0 at the start), o = S^T q / (max(|n.q|, e^-m) +
+    1e-6).  q times dim^-1/2; i = cap tanh((W_i h + b_i) / cap), f = log sigmoid(cap tanh((W_f h + b_f) / cap)), one number per
+    head and token each.  Every head's output is divided by its root mean square; all heads times a weight vector, times
+    sigmoid of a gate projection."""
+    heads: int
+    dim: int
+    vdim: int
+    gate_cap: float
+
+    kind = "mlstm"
+    kv_heads = 0
+    chunk = 0
+    window = 0
+    keep_first = 0
+    pool = 0
+
+    @property
+    def proj_cols(self) -> int:
+        """columns of the fused projection [q | k | v | gate | i | f]"""
+        return 2 * self.heads * self.dim + 2 * self.heads * self.vdim + 2 * self.heads
+
+    @property
+    def attn_cols(self) -> int:
+        return self.heads * self.vdim
+
+    def cache_shape(self) -> tuple[int, int, int]:
+        return (0, 0, 0)                 # no cache pages
+
+    @property
+    def state_shapes(self) -> tuple:
+        """S, n and m"""
+        return (self.heads * self.dim * self.vdim, self.heads * self.dim, self.heads)
+
+
+@dataclass(frozen=True)
 class ParallelMixerSpec:
     """Two mixers side by side on the same input (an attention mixer with cache pages and a mixer with a state).  `join`
     "sum": left_scale * left + right_scale * right, one output projection over both sides' heads; "rms_mean": each side has
@@ -460,6 +511,10 @@ class ParallelMixerSpec:
     @property
     def keep_first(self) -> int:
         return self.left.keep_first
+
+    @property
+    def pool(self) -> int:
+        return self.left.pool
 
     @property
     def proj_cols(self) -> int:
@@ -529,6 +584,7 @@ class LatentMixerSpec:
 @dataclass(frozen=True)
 class DenseSpec:
     """Gated dense feed-forward: g = W_gate h, u = W_up h, output W_down act(g, u).  activation "silu": silu(g) u;
+    "gelu_tanh": gelu(g) u with the tanh form;
     "clamped_swish": g <- min(g, limit), u <- clamp(u, -limit, limit), g sigmoid(alpha g) (u + 1).  "relu2" has no gate:
     W_down max(W_up h, 0)^2.  "polynorm" has no gate either: W_down (a N(z) + b N(z^2) + c N(z^3) + e) with z = W_up h,
     powers element by element, N = division by the root mean square over the ff values, and four learned numbers."""
@@ -550,7 +606,9 @@ class MoESpec:
     "biased": softmax over experts + identity router outputs, the `top` largest of score + a stored correction are chosen,
     the weights are the scores themselves (`renorm` False) -- the last `identity` outputs stand for experts that return
     their input and have no matrices; `shared_gate`: the shared expert's output is multiplied by sigmoid of one more
-    projection, a number per token."""
+    projection, a number per token.  Router "logits": logits + a stored bias, the `top` largest are chosen, weights = softmax
+    over the chosen ones alone.  `activation` "silu": experts with a gate, W_down (silu(W_gate h) * W_up h); "gelu": without,
+    W_down gelu(W_up h) with the erf form (the shared expert alike)."""
     experts: int
     top: int
     ff: int
@@ -561,8 +619,20 @@ class MoESpec:
     identity: int = 0
     renorm: bool = True
     shared_gate: bool = False
+    activation: str = "silu"
 
     kind = "moe"
+
+    @property
+    def shared_slot(self) -> bool:
+        """A shared expert without a gate of its own that is no wider than the experts rides in their stack (padded with zero
+        rows) as one more matrix that every token takes with weight 1."""
+        return self.router == "logits" and 0 < self.shared_ff <= self.ff
+
+    @property
+    def slots(self) -> int:
+        """(token, expert) rows per token"""
+        return self.top + (1 if self.shared_slot else 0)
 
     @property
     def routes(self) -> int:
@@ -572,7 +642,8 @@ class MoESpec:
 
 @dataclass(frozen=True)
 class LayerSpec:
-    mixer: "AttentionMixerSpec | LatentMixerSpec | LinearMixerSpec | GatedLinearMixerSpec | DeltaMixerSpec | ParallelMixerSpec"
+    mixer: ("AttentionMixerSpec | LatentMixerSpec | LinearMixerSpec | GatedLinearMixerSpec | DeltaMixerSpec | MatrixLSTMSpec | "
+            "ParallelMixerSpec")
     mlp: "MoESpec | DenseSpec | None"
 
 
@@ -587,11 +658,12 @@ class LayeredConfig:
     norm_eps: float = 1e-5
     logit_scale: float = 1.0
     logit_softcap: float = 0.0
-    # block form: "post_norm" x += LN(sublayer(x)) twice; "parallel" h = norm(x), x += s1 mixer(h) + s2 ff(h);
+    # block form: "post_norm" x += norm(sublayer(x)) twice (with layer_scale: x += s * norm(sublayer(x))); "parallel" h = norm(x), x += s1 mixer(h) + s2 ff(h);
     # "pre_norm" x += m mixer(c1(norm1(x))), x += m ff(c2(norm2(x))) with m = residual_mult and c the input convolution;
     # "sandwich" x += norm1b(mixer(norm1(x))), x += norm2b(ff(norm2(x)))
     block: str = "post_norm"
-    # "layernorm" (weight + bias), "layernorm_nobias", "rmsnorm_1p" (x / rms * (1 + w)) or "dyt" (tanh(alpha x) * w + b)
+    # "layernorm" (weight + bias), "layernorm_nobias", "rmsnorm" (x / rms * w), "rmsnorm_1p" (x / rms * (1 + w)) or "dyt"
+    # (tanh(alpha x) * w + b)
     norm: str = "layernorm"
     tied_head: bool = False            # the logits are products with the embedding table
     residual_mult: float = 1.0         # pre_norm blocks: factor on every sublayer's result before it joins the residual
@@ -830,9 +902,67 @@ def _sumitar_config(d: dict) -> LayeredConfig:
                          norm_eps=float((d.get("norm") or {}).get("eps", 1e-6)), block="sandwich", norm="dyt", tied_head=True)
 
 
+def _vosolorn_config(d: dict) -> LayeredConfig:
+    """Vosolorn: blocks with an RMS norm on each sublayer's output and a layer scale behind it, an RMS norm on the embedding;
+    two mixers -- "attention" (q / k norm in front of a rotation in pairs, rotated values, a sliding window with pooled blocks
+    before it) and "mlstm" (the matrix memory of xLSTM) -- and two feed-forwards (gated with the tanh form of gelu, or experts
+    without gates behind a router that chooses and weighs by its logits, with a shared expert); the logits are scaled products
+    with the embedding table.  What the design fixes is set here; sizes and constants come from the file."""
+
+    def sizes(m, where):
+        heads, dim = int(m["heads"]), int(m["dim"])
+        kv = int(m.get("kv_heads") or heads)
+        vdim = int(m.get("vdim") or dim)
+        if heads < 1 or dim < 1 or vdim < 1 or kv < 1 or heads % kv:
+            raise ValueError(f"{where}: {heads} heads over {kv} key/value heads")
+        return heads, kv, dim, vdim
+
+    layers = []
+    for i, L in enumerate(d["layers"]):
+        m, kind, where = L["mixer"], L.get("type"), f"Vosolorn: layer {i}"
+        heads, kv, dim, vdim = sizes(m, where)
+        if kind == "attention":
+            mask = m.get("mask") or {}
+            window = int(mask.get("size") or 0)
+            rot = _rotary(m.get("rot"), dim, where)
+            if rot is None:
+                raise ValueError(f"{where}: attention without a rotation")
+            if vdim % 2:
+                raise ValueError(f"{where}: values of {vdim} elements cannot turn in pairs")
+            pool = int(mask.get("pool") or 0) if window > 0 else 0          # no window: every token is seen itself
+            if window < 0 or pool < 0:
+                raise ValueError(f"{where}: window {window}, blocks of {pool}")
+            mixer = AttentionMixerSpec(heads=heads, kv_heads=kv, dim=dim, vdim=vdim, scale=float(m["scale"]), window=window, pool=pool,
+                                       qk_norm=True, norm_first=True, out_gate=False, distance_bias=False, rot_values=True,
+                                       rot=RotarySpec(rot.dims, rot.base, rot.factor, layout="pairs"))
+        elif kind == "mlstm":
+            mixer = MatrixLSTMSpec(heads=heads, dim=dim, vdim=vdim, gate_cap=float(m["gate_cap"]))
+            if mixer.gate_cap <= 0:
+                raise ValueError(f"{where}: gate cap {mixer.gate_cap}")
+        else:
+            raise ValueError(f"{where} has unknown type {kind!r}")
+        mlp = None
+        f = L.get("mlp")
+        if f:
+            if f.get("kind") == "dense":
+                mlp = DenseSpec(ff=int(f["ff"]), activation="gelu_tanh")
+            elif f.get("kind") == "moe":
+                r = f["router"]
+                mlp = MoESpec(experts=int(r["experts"]), top=int(r["top"]), ff=int(f["expert"]["ff"]),
+                              shared_ff=int((f.get("shared") or {}).get("ff") or 0), router="logits", activation="gelu")
+                if not 1 <= mlp.top <= mlp.experts:
+                    raise ValueError(f"{where}: top {mlp.top} of {mlp.experts} experts")
+            else:
+                raise ValueError(f"{where} has unknown feed-forward kind {f.get('kind')!r}")
+        layers.append(LayerSpec(mixer, mlp))
+    return LayeredConfig(architecture="Vosolorn", vocab_size=int(d["vocab"]), hidden_size=int(d["width"]), layers=layers,
+                         norm_eps=float((d.get("norm") or {}).get("eps", 1e-6)), logit_scale=float(d.get("logit_scale", 1.0)),
+                         block="post_norm", norm="rmsnorm", embed_norm=True, layer_scale=True, tied_head=True)
+
+
 # config.json "architecture" -> parser (the model registry of the layered families)
 LAYERED_ARCHITECTURES = {"dolurax": _dolurax_config, "turutar": _turutar_config, "rezulorn": _rezulorn_config,
-                         "sumitar": _sumitar_config}
+                         "sumitar": _sumitar_config, "vosolorn": _vosolorn_config}
 
 
 def layered_config_from_json(d: dict) -> LayeredConfig | None:
@@ -843,5 +973,5 @@ def layered_config_from_json(d: dict) -> LayeredConfig | None:
 
 __all__ = ["ModelSpec", "TransformerConfig", "GPT2Config", "LlamaConfig", "Qwen3Config", "GPT2_SPEC", "LLAMA_SPEC",
            "QWEN2_SPEC", "QWEN3_SPEC", "QWEN3_MOE_SPEC", "MIXTRAL_SPEC", "MODEL_SPECS", "detect_model_spec",
-           "named_config", "AttentionMixerSpec", "LatentMixerSpec", "RotarySpec", "LinearMixerSpec", "GatedLinearMixerSpec", "DeltaMixerSpec", "ParallelMixerSpec", "DenseSpec", "MoESpec", "LayerSpec", "LayeredConfig",
+           "named_config", "AttentionMixerSpec", "LatentMixerSpec", "RotarySpec", "LinearMixerSpec", "GatedLinearMixerSpec", "DeltaMixerSpec", "MatrixLSTMSpec", "ParallelMixerSpec", "DenseSpec", "MoESpec", "LayerSpec", "LayeredConfig",
            "LAYERED_ARCHITECTURES", "layered_config_from_json"]

@@ -6,6 +6,7 @@ from .gated_recurrent import DeltaRuleMixer, GatedLinearMixer
 from .linear_attention import LinearAttentionMixer, ParallelMixer
 from .latent_attention import LatentAttentionMixer
 from .token_side import TokenSideInput
+from .matrix_lstm import MatrixLSTMMixer
 from .linear import Linear, LinearBF16, LinearFP8, LinearNVF4, LinearRows, interleave_gate_up
 from .mlp import MLP
 from .moe import MoELayer
@@ -16,5 +17,5 @@ from .rope import apply_rotary_pos_emb_numpy, precompute_freqs_cis
 
 __all__ = ["Attention", "TransformerBlock", "Linear", "LinearBF16", "LinearFP8", "LinearNVF4", "MLP", "MoELayer",
            "Norm", "RowNorm", "CausalConvRows", "PostNormBlock", "ParallelBlock", "PreNormBlock", "SandwichBlock", "GatedDenseRows", "SquaredReluRows", "PolyNormRows",
-           "GatedLinearMixer", "DeltaRuleMixer", "BiasedRouterMoE",
+           "GatedLinearMixer", "DeltaRuleMixer", "BiasedRouterMoE", "MatrixLSTMMixer",
            "LinearAttentionMixer", "ParallelMixer", "LatentAttentionMixer", "TokenSideInput", "LinearRows", "interleave_gate_up", "GroupedRouterMoE", "PagedAttentionMixer", "apply_rotary_pos_emb_numpy", "precompute_freqs_cis"]

@@ -9,7 +9,8 @@ from .attention import Attention
 from .linear import can_fuse_norm
 from .mlp import MLP
 from .moe import MoELayer
-from .norm import Norm
+from .moe_rows import GroupedRouterMoE
+from .norm import Norm, RowNorm
 
 
 class TransformerBlock:
@@ -79,38 +80,66 @@ class TransformerBlock:
 
 
 class PostNormBlock:
-    """Block of the token-major models with the norm on the sublayer's OUTPUT: x += LN1(mixer(x)), then
-    x += LN2(ff(x)); both sublayers read the float32 residual stream itself.  Each "norm + add" is one launch that
-    also folds the feed-forward's weighted expert sum and shared expert (pgk_combine_layernorm_f32)."""
+    """Block of the token-major models with the norm on the sublayer's OUTPUT: x += norm1(mixer(x)), then
+    x += norm2(ff(x)); both sublayers read the float32 residual stream itself.  Each "norm + add" is one launch that
+    also folds the feed-forward's weighted expert sum and shared expert: pgk_combine_layernorm_f32 for a LayerNorm (a weight and
+    a bias), pgk_rms_join_f32 for an RMS norm (a `RowNorm`; a per-channel factor behind the norm is part of its weight).
+    Per-sequence state of the block in the cache manager: whatever the mixer keeps."""
 
-    def __init__(self, mixer, norm1: tuple[GPUArray, GPUArray], mlp, norm2: "tuple[GPUArray, GPUArray] | None", eps: float):
+    def __init__(self, mixer, norm1: "tuple[GPUArray, GPUArray] | RowNorm", mlp, norm2: "tuple[GPUArray, GPUArray] | RowNorm | None",
+                 eps: float):
         self.mixer, self.mlp = mixer, mlp
         self.norm1, self.norm2, self.eps = norm1, norm2, float(eps)
+        for n in (norm1, norm2):
+            if isinstance(n, RowNorm) and (n.kind != "rmsnorm" or n.offset != 0.0):
+                raise ValueError("PostNormBlock: a LayerNorm pair or an RMS norm with a plain weight")
+        if (mlp is None) != (norm2 is None):
+            raise ValueError("PostNormBlock: a feed-forward comes with its norm")
+
+    @property
+    def state_shapes(self) -> tuple:
+        return tuple(self.mixer.spec.state_shapes)
 
     norm = None                          # no norm in front of the block: nothing for the block before to fuse with
 
     def forward(self, ctx, x: GPUArray, cache_index: int | None = None, add_ptr: int | None = None, normed: bool = False,
                 next_norm=None, next_add_ptr: int | None = None) -> bool:
-        from ..._lib import api
-        from ...core.stream import current_stream_handle as _st
         if add_ptr is not None:
             raise ValueError("PostNormBlock: no loop passes in this block form")
         T, W = ctx.T, x.shape[1]
         y = ctx.buf.y
-        self.mixer.forward(ctx, x, y, cache_index)
-        api.combine_layernorm_f32(y.device_ptr, None, None, None, None, 0, self.norm1[0].device_ptr,
-                                  self.norm1[1].device_ptr, self.eps, x.device_ptr, T, W, 1, _st())
-        if self.mlp is not None:
+        if self.state_shapes:
+            self.mixer.forward(ctx, x, y, cache_index, state=ctx.cache.state[cache_index])
+        else:
+            self.mixer.forward(ctx, x, y, cache_index)
+        self._join(y.device_ptr, None, None, None, 0, self.norm1, x, T, W)
+        if self.mlp is None:
+            return False
+        if isinstance(self.mlp, GroupedRouterMoE):
             base, parts, inv, wts, top = self.mlp.forward(ctx, x, y)
-            api.combine_layernorm_f32(base, None, parts, inv, wts, top, self.norm2[0].device_ptr,
-                                      self.norm2[1].device_ptr, self.eps, x.device_ptr, T, W, 1, _st())
+        else:                                            # a dense feed-forward: plain rows
+            self.mlp.forward(ctx, x.device_ptr, y.device_ptr)
+            base, parts, inv, wts, top = y.device_ptr, None, None, None, 0
+        self._join(base, parts, inv, wts, top, self.norm2, x, T, W)
         return False
+
+    def _join(self, base, parts, inv, wts, top: int, norm, x: GPUArray, T: int, W: int) -> None:
+        """x += norm(base + weighted expert rows)"""
+        from ..._lib import api
+        from ...core.stream import current_stream_handle as _st
+        if isinstance(norm, RowNorm):
+            api.rms_join_f32(base, parts, inv, wts, top, norm.weight.device_ptr, norm.eps, x.device_ptr, T, W, _st())
+        else:
+            api.combine_layernorm_f32(base, None, parts, inv, wts, top, norm[0].device_ptr, norm[1].device_ptr, self.eps, x.device_ptr,
+                                      T, W, 1, _st())
 
     @property
     def weight_bytes(self) -> int:
-        n = self.mixer.weight_bytes + 2 * self.norm1[0].nbytes
+        def size(norm):
+            return norm.nbytes if isinstance(norm, RowNorm) else 2 * norm[0].nbytes
+        n = self.mixer.weight_bytes + size(self.norm1)
         if self.mlp is not None:
-            n += self.mlp.weight_bytes + 2 * self.norm2[0].nbytes
+            n += self.mlp.weight_bytes + size(self.norm2)
         return n
 
 

@@ -3,6 +3,7 @@ a time, and `GroupedRouterMoE`).  Two launches: the fused gate/up product whose 
 interleaved (gate_j, up_j) pairs, and the down projection.
 
   activation "silu":           silu(g) * u
+  activation "gelu_tanh":      gelu(g) * u, the tanh form
   activation "clamped_swish":  g <- min(g, limit), u <- clamp(u, -limit, limit), g * sigmoid(alpha g) * (u + 1)
 
 `SquaredReluRows` is the feed-forward without a gate, W_down max(W_up h, 0)^2, the activation again in the first product's
@@ -19,7 +20,7 @@ from .linear import LinearRows
 
 class GatedDenseRows:
     def __init__(self, spec: DenseSpec, gate_up: LinearRows, down: LinearRows):
-        if spec.activation not in ("silu", "clamped_swish"):
+        if spec.activation not in ("silu", "gelu_tanh", "clamped_swish"):
             raise ValueError(f"GatedDenseRows: unknown activation {spec.activation!r}")
         if gate_up.out_features != 2 * spec.ff or down.in_features != spec.ff:
             raise ValueError("GatedDenseRows: matrices do not match the feed-forward size")
@@ -32,8 +33,8 @@ class GatedDenseRows:
     def forward(self, ctx, h_ptr: int, out_ptr: int, out_scale: int | None = None) -> None:
         sp, T = self.spec, ctx.T
         W, act = self.gate_up.in_features, ctx.buf.shared_act
-        if sp.activation == "silu":
-            self.gate_up.forward_seq(h_ptr, W, T, act.device_ptr, sp.ff, epilogue=1)
+        if sp.activation in ("silu", "gelu_tanh"):
+            self.gate_up.forward_seq(h_ptr, W, T, act.device_ptr, sp.ff, epilogue=1 if sp.activation == "silu" else 7)
         else:
             self.gate_up.forward_seq(h_ptr, W, T, act.device_ptr, sp.ff, epilogue=3, p0=sp.alpha, p1=sp.limit)
         if out_scale is None:

@@ -246,7 +246,8 @@ class LinearRows:
     """Linear layer of the token-major models (net-new): float32 activations [rows, K], weights [N, K] (or a stack
     [E, N, K] of expert matrices) in bfloat16 or float32, float32 accumulation and output.  Many rows run as tiled
     GEMMs (tensor cores for bfloat16 weights), up to eight rows through the streaming few-row kernel.  epilogue:
-    0 plain, 1 gate/up pairs -> silu(gate) * up (rows of W interleaved by `interleave_gate_up`), 2 scale + tanh cap;
+    0 plain, 1 gate/up pairs -> silu(gate) * up (rows of W interleaved by `interleave_gate_up`), 2 scale + tanh cap,
+    7 gate/up pairs -> gelu_tanh(gate) * up, 8 gelu (erf form) of the product;
     `forward_seq` adds 3 clamped gate/up pairs, 4 scaled accumulation into the output, 5 gelu * gathered table entry,
     and batches of per-head products."""
 
@@ -266,7 +267,7 @@ class LinearRows:
 
     @property
     def out_cols(self) -> int:
-        return self.out_features // 2 if self.epilogue == 1 else self.out_features
+        return self.out_features // 2 if self.epilogue in (1, 7) else self.out_features
 
     @property
     def nbytes(self) -> int:

@@ -24,13 +24,24 @@ from .linear import LinearRows
 
 
 class GroupedRouterMoE:
+    """With spec.router "logits" the route launch is pgk_moe_route_logits (a bias on the logits, softmax over the chosen ones), and
+    a shared expert no wider than the others may ride in their stack as the last matrix, which every token takes with weight 1
+    (spec.shared_slot): no launches of its own.  Experts without gates put the up matrices in `gate_up` with their activation's
+    epilogue."""
+
     def __init__(self, spec: MoESpec, router: GPUArray, gate_up: LinearRows, down: LinearRows,
-                 shared_gate_up: LinearRows | None = None, shared_down: LinearRows | None = None):
-        self.spec, self.router = spec, LinearRows(router)
+                 shared_gate_up: LinearRows | None = None, shared_down: LinearRows | None = None,
+                 router_bias: GPUArray | None = None):
+        self.spec, self.router, self.router_bias = spec, LinearRows(router), router_bias
         self.gate_up, self.down = gate_up, down
         self.shared_gate_up, self.shared_down = shared_gate_up, shared_down
-        if gate_up.groups != spec.experts or down.groups != spec.experts:
+        self.stack = spec.experts + (1 if spec.shared_slot else 0)
+        if gate_up.groups != self.stack or down.groups != self.stack:
             raise ValueError("GroupedRouterMoE: expert stacks do not match the router")
+        if spec.router not in ("grouped", "logits") or (router_bias is not None and spec.router != "logits"):
+            raise ValueError(f"GroupedRouterMoE: router {spec.router!r}")
+        if spec.shared_slot and shared_gate_up is not None:
+            raise ValueError("GroupedRouterMoE: the shared expert rides in the stack")
 
     @property
     def weight_bytes(self) -> int:
@@ -43,12 +54,17 @@ class GroupedRouterMoE:
         """Returns (base, parts, inv, weights, top) for the combine + norm launch: base = the shared expert's output
         rows (or None), parts [T * top, W] the routed experts' outputs, inv [T, top] their rows."""
         sp, T, b = self.spec, ctx.T, ctx.buf
-        W, top, ff = self.gate_up.in_features, sp.top, sp.ff
+        W, top, ff = self.gate_up.in_features, sp.slots, sp.ff
         few = T <= LinearRows.FEW
         self.router.forward(x.device_ptr, W, T, b.moe_z.device_ptr, sp.experts)       # float32 logits [T, E]
-        api.moe_route_grouped(b.moe_z.device_ptr, sp.experts, T, sp.experts, top,
-                              sp.group_count, sp.group_keep, b.moe_idx.device_ptr, b.moe_w.device_ptr,
-                              None if few else b.moe_rank.device_ptr, None if few else b.moe_counts.device_ptr, _st())
+        rank, counts = (None, None) if few else (b.moe_rank.device_ptr, b.moe_counts.device_ptr)
+        if sp.router == "logits":
+            api.moe_route_logits(b.moe_z.device_ptr, sp.experts, T, sp.experts, sp.top,
+                                 self.router_bias.device_ptr if self.router_bias is not None else None,
+                                 sp.experts if sp.shared_slot else -1, b.moe_idx.device_ptr, b.moe_w.device_ptr, rank, counts, _st())
+        else:
+            api.moe_route_grouped(b.moe_z.device_ptr, sp.experts, T, sp.experts, top, sp.group_count, sp.group_keep,
+                                  b.moe_idx.device_ptr, b.moe_w.device_ptr, rank, counts, _st())
         if few:
             slot_tok, iota = ctx.slot_rows(top)
             self.gate_up.forward_per_row(x.device_ptr, W, T * top, b.moe_act.device_ptr, ff, slot_tok, b.moe_idx.device_ptr)
@@ -56,7 +72,7 @@ class GroupedRouterMoE:
             inv = iota
         else:
             api.moe_row_lists(b.moe_counts.device_ptr, b.moe_off.device_ptr, b.moe_idx.device_ptr, b.moe_rank.device_ptr,
-                              b.moe_perm.device_ptr, b.moe_inv.device_ptr, sp.experts, T, top, _st())
+                              b.moe_perm.device_ptr, b.moe_inv.device_ptr, self.stack, T, top, _st())
             self.gate_up.forward_grouped(x.device_ptr, W, b.moe_act.device_ptr, ff, b.moe_perm.device_ptr,
                                          b.moe_off.device_ptr, T)
             self.down.forward_grouped(b.moe_act.device_ptr, ff, b.moe_parts.device_ptr, W, None, b.moe_off.device_ptr, T)

@@ -16,6 +16,11 @@ launch, pgk_seq_mixer_prep_rot.  Kept first positions under a window, the logari
 head) and sigmoid weights without normalisation (a learned number per head added to the score) are arguments of the
 attention launch as well.  `attend` is the mixer without its two matrix products: it runs on a block of columns of a wider
 fused projection, which is how a mixer that runs beside another one shares their products.
+
+The rotation may pair neighbours instead of halves, follow the q / k norm instead of preceding it, and take the values along
+(the attention launch then turns the heads' outputs back).  With pooled blocks the preparation also leaves the means of every
+finished block's keys and values (a launch of its own behind it unless every sequence brings one token), and the attention
+launch reads those rows for everything that lies before the window.
 """
 from __future__ import annotations
 
@@ -30,12 +35,12 @@ from .linear import LinearRows
 
 
 def key_slices(ctx, heads: int, kv_heads: int, chunk: int, window: int, queries_per_tile: int, heads_per_block: int,
-               decode_heads_per_block: int, keep_first: int = 0) -> int:
+               decode_heads_per_block: int, keep_first: int = 0, pool: int = 0) -> int:
     """Few long tiles (decoding over a long context): the key range of every tile is cut into this many slices so that the
     whole GPU reads the cache.  A power of two, so that a decode step's launch shapes change rarely."""
     n_tiles = ctx.tiles(queries_per_tile)[1]
     rep = heads // kv_heads
-    keys = ctx.max_keys(chunk, window, keep_first)
+    keys = ctx.max_keys(chunk, window, keep_first, pool)
     if ctx.decode_only:          # the decoding kernel: eight warps take 32 keys each per round
         blocks = n_tiles * kv_heads * -(-rep // decode_heads_per_block)
         want = max(1, min(64, -(-keys // 256), 592 // max(1, blocks)))
@@ -82,6 +87,12 @@ class PagedAttentionMixer:
             raise ValueError(f"layer {layer}: the logarithmic distance term and its two vectors do not agree")
         if s.keep_first and (s.window <= 0 or s.chunk):
             raise ValueError(f"layer {layer}: kept first positions need a window and no chunks")
+        if s.pool and (s.window <= 0 or s.chunk or s.keep_first or s.distance_bias):
+            raise ValueError(f"layer {layer}: pooled blocks need a window, no chunks, no kept positions and no distance term")
+        if (s.rot_values or s.norm_first) and s.rot is None:
+            raise ValueError(f"layer {layer}: rotated values and a norm in front of the rotation need a rotation")
+        if s.rot_values and s.vdim % 2:
+            raise ValueError(f"layer {layer}: values of {s.vdim} elements cannot turn in pairs")
         # the preparation launch with rotation / unweighted norm / no norm
         self.rot_prep = s.rot is not None or not s.qk_norm or not s.norm_weight
         if s.qkv_bias != (q_bias is not None and k_bias is not None and v_bias is not None) and not s.qk_bias:
@@ -97,6 +108,8 @@ class PagedAttentionMixer:
             raise ValueError(f"layer {layer}: the q / k norm needs its weights")
         self.norm_mode = 0 if not s.qk_norm else (2 if s.norm_weight else 1)
         self.inv_freq = from_numpy(np.asarray(s.rot.inv_freq(), np.float64)) if s.rot is not None else None
+        self.v_inv_freq = from_numpy(np.asarray(s.rot.value_inv_freq(s.vdim), np.float64)) if s.rot_values else None
+        self.pairs = 1 if s.rot is not None and s.rot.layout == "pairs" else 0
         self.distance, self.weight_bias, self.out_mult = distance, weight_bias, float(out_mult)
         self.q_cols, self.k_cols = s.heads * s.dim, s.kv_heads * s.dim
         self.v_cols = s.kv_heads * s.vdim if s.values == "own" else 0
@@ -120,7 +133,7 @@ class PagedAttentionMixer:
     def key_slices(self, ctx) -> int:
         s = self.spec
         return key_slices(ctx, s.heads, s.kv_heads, s.chunk, s.window, self.queries_per_tile, self.heads_per_block,
-                          self.decode_heads_per_block, s.keep_first)
+                          self.decode_heads_per_block, s.keep_first, s.pool)
 
     def forward(self, ctx, x: GPUArray, out: GPUArray, cache_index: int | None = None, out_scale: int | None = None,
                 state=None) -> None:
@@ -149,12 +162,16 @@ class PagedAttentionMixer:
         kc, vc = cache.k[ci], cache.v[ci]
         if self.rot_prep:
             bias = [b.device_ptr if (s.qkv_bias and b is not None) else None for b in (self.q_bias, self.k_bias, self.v_bias)]
-            api.seq_mixer_prep_rot_ex(proj_ptr, ld, T, s.heads, s.kv_heads, s.dim, s.vdim, 0, self.q_cols, self.q_cols + self.k_cols,
+            pool = cache.pool_rows(ci) and s.pool
+            pk, pv = (cache.pk[ci].device_ptr, cache.pv[ci].device_ptr) if pool else (None, None)
+            api.seq_mixer_prep_rot_ex2(proj_ptr, ld, T, s.heads, s.kv_heads, s.dim, s.vdim, 0, self.q_cols, self.q_cols + self.k_cols,
                                       s.rot.dims if s.rot is not None else 0,
                                       self.inv_freq.device_ptr if self.inv_freq is not None else None, self.norm_mode,
                                       self.q_norm.device_ptr if self.q_norm is not None else None,
                                       self.k_norm.device_ptr if self.k_norm is not None else None, self.eps, bias[0], bias[1],
-                                      bias[2], self.head_temp.device_ptr if self.head_temp is not None else None, kc.device_ptr,
+                                      bias[2], self.head_temp.device_ptr if self.head_temp is not None else None, self.pairs,
+                                      1 if s.norm_first else 0, self.v_inv_freq.device_ptr if s.rot_values else None, pool,
+                                      cache.pool_rows(ci), pk, pv, 1 if ctx.decode_only else 0, kc.device_ptr,
                                       vc.device_ptr, cache.dtype_code, cache.table_dev.device_ptr, cache.pool.max_pages,
                                       cache.page_size, ctx.slot_ptr, ctx.pos_ptr, _st())
         elif s.norm_scope == "all":
@@ -176,15 +193,17 @@ class PagedAttentionMixer:
             ws = ctx.workspace(T * s.heads * splits * (s.vdim + 2)).device_ptr
             tickets = ctx.buf.tickets.device_ptr
         gate_mode = 0 if not s.out_gate else (2 if s.gate_per_head else 1)
-        api.seq_attention_ex2(proj_ptr, ld, 0, proj_ptr, ld, self.q_cols + self.k_cols + self.v_cols, gate_mode,
+        api.seq_attention_ex3(proj_ptr, ld, 0, proj_ptr, ld, self.q_cols + self.k_cols + self.v_cols, gate_mode,
                               attn_ptr, ldo, kc.device_ptr, vc.device_ptr, s.dim, s.vdim, cache.dtype_code,
                               cache.table_dev.device_ptr, cache.pool.max_pages, cache.page_size, tiles_ptr, n_tiles,
                               self.slopes.device_ptr if self.slopes is not None else None,
                               self.slopes2.device_ptr if self.slopes2 is not None else None,
                               self.sinks.device_ptr if self.sinks is not None else None, s.heads, s.kv_heads, s.dim, s.vdim,
                               s.chunk, s.window, s.keep_first, s.scale, s.softcap, 1 if s.weights == "sigmoid" else 0,
-                              self.weight_bias.device_ptr if self.weight_bias is not None else None, self.out_mult, splits, ws,
-                              tickets, 1 if ctx.decode_only else 0, _st())
+                              self.weight_bias.device_ptr if self.weight_bias is not None else None, self.out_mult, s.pool,
+                              cache.pool_rows(ci), cache.pk[ci].device_ptr if s.pool else None,
+                              cache.pv[ci].device_ptr if s.pool else None, self.v_inv_freq.device_ptr if s.rot_values else None,
+                              self.pairs, splits, ws, tickets, 1 if ctx.decode_only else 0, _st())
 
 
 __all__ = ["PagedAttentionMixer", "key_slices"]

@@ -31,6 +31,12 @@ l<i>.mix.right.{q,f,v,o}, .right.f.b, .right.lower, .right.norm [vdim], .right.o
 l<i>.mlp.{up,down,act}; experts l<i>.mlp.e<j>.{gate,up,down}, .router [experts + identity, width], .correction,
 .shared.{gate,up,down,sg}.  Both sides' projections of a parallel mixer are one matrix ([left q | k | v | right q | f | v]), a
 delta mixer's are [q | k | v | g | b | a]; the router matrix carries the shared expert's gate row as its last row.
+
+Vosolorn tensor names: embed (also the head), embed.norm, final.norm; per layer l<i>.norm1, norm2, ls1, ls2; "attention"
+l<i>.mix.{q,k,v,o}, .q.norm, .k.norm [dim]; "mlstm" l<i>.mix.{q,k,v,g,o}, .norm [heads x vdim], .i, .f [heads, width] with .i.b,
+.f.b; dense feed-forward l<i>.mlp.{gate,up,down}; experts l<i>.mlp.e<j>.{up,down}, .router [experts, width] with .router.b,
+.shared.{up,down}.  An mLSTM mixer's projections are one matrix [q | k | v | g | i | f]; a layer scale multiplies the weight of the
+norm in front of it; a shared expert no wider than the others is the last matrix of their stack.
 """
 from __future__ import annotations
 
@@ -49,6 +55,7 @@ from .layers.gated_recurrent import DeltaRuleMixer, GatedLinearMixer
 from .layers.linear_attention import LinearAttentionMixer, ParallelMixer
 from .layers.latent_attention import LatentAttentionMixer
 from .layers.linear import LinearRows, interleave_gate_up
+from .layers.matrix_lstm import MatrixLSTMMixer
 from .layers.moe_rows import BiasedRouterMoE, GroupedRouterMoE
 from .layers.norm import CausalConvRows, RowNorm
 from .layers.paged_attention import PagedAttentionMixer
@@ -317,8 +324,62 @@ def _build_sumitar(config: LayeredConfig, t: _Tensors, dtype: str) -> LayeredCau
     return LayeredCausalModel(config, embed, blocks, norm("final.norm"), LinearRows(embed), dtype)
 
 
+def _build_vosolorn(config: LayeredConfig, t: _Tensors, dtype: str) -> LayeredCausalModel:
+    W, V, eps = config.hidden_size, config.vocab_size, config.norm_eps
+
+    def norm(name, scale=None):               # the factor behind a norm is part of its weight
+        w = t.f32(name, (W,))
+        return RowNorm("rmsnorm", _vector(w if scale is None else w * t.f32(scale, (W,))), None, eps)
+
+    blocks = []
+    for i, L in enumerate(config.layers):
+        p, m = f"l{i}.", L.mixer
+        mp = p + "mix."
+        H, D, Dv = m.heads, m.dim, m.vdim
+        o_proj = LinearRows(_matrix(t.f32(mp + "o", (W, H * Dv)), dtype))
+        if m.kind == "attention":
+            fused = np.concatenate([t.f32(mp + "q", (H * D, W)), t.f32(mp + "k", (m.kv_heads * D, W)),
+                                    t.f32(mp + "v", (m.kv_heads * Dv, W))])
+            mixer = PagedAttentionMixer(m, i, LinearRows(_matrix(fused, dtype)), o_proj, _vector(t.f32(mp + "q.norm", (D,))),
+                                        _vector(t.f32(mp + "k.norm", (D,))), eps)
+        else:
+            fused = np.concatenate([t.f32(mp + "q", (H * D, W)), t.f32(mp + "k", (H * D, W)), t.f32(mp + "v", (H * Dv, W)),
+                                    t.f32(mp + "g", (H * Dv, W)), t.f32(mp + "i", (H, W)), t.f32(mp + "f", (H, W))])
+            mixer = MatrixLSTMMixer(m, i, LinearRows(_matrix(fused, dtype)), o_proj, _vector(t.f32(mp + "i.b", (H,))),
+                                    _vector(t.f32(mp + "f.b", (H,))), _vector(t.f32(mp + "norm", (H * Dv,))), eps)
+        mlp = norm2 = None
+        f = L.mlp
+        if f is not None:
+            q = p + "mlp."
+            norm2 = norm(p + "norm2", p + "ls2")
+            if f.kind == "dense":
+                gu = interleave_gate_up(t.f32(q + "gate", (f.ff, W)), t.f32(q + "up", (f.ff, W)))
+                mlp = GatedDenseRows(f, LinearRows(_matrix(gu, dtype)), LinearRows(_matrix(t.f32(q + "down", (W, f.ff)), dtype)))
+            else:
+                up = [t.f32(f"{q}e{e}.up", (f.ff, W)) for e in range(f.experts)]
+                dn = [t.f32(f"{q}e{e}.down", (W, f.ff)) for e in range(f.experts)]
+                sup = sdn = None
+                if f.shared_ff:
+                    su, sd = t.f32(q + "shared.up", (f.shared_ff, W)), t.f32(q + "shared.down", (W, f.shared_ff))
+                    if f.shared_slot:
+                        pad = f.ff - f.shared_ff
+                        up.append(np.pad(su, ((0, pad), (0, 0))))
+                        dn.append(np.pad(sd, ((0, 0), (0, pad))))
+                    else:
+                        sup, sdn = LinearRows(_matrix(su, dtype), epilogue=8), LinearRows(_matrix(sd, dtype))
+                # the router stays float32 in both modes: its logits come from the unrounded residual stream
+                mlp = GroupedRouterMoE(f, _matrix(t.f32(q + "router", (f.experts, W)), "float32"),
+                                       LinearRows(_matrix(np.stack(up), dtype), epilogue=8), LinearRows(_matrix(np.stack(dn), dtype)),
+                                       sup, sdn, router_bias=_vector(t.f32(q + "router.b", (f.experts,))))
+        blocks.append(PostNormBlock(mixer, norm(p + "norm1", p + "ls1"), mlp, norm2, eps))
+    embed = _matrix(t.f32("embed", (V, W)), dtype)
+    head = LinearRows(embed, epilogue=2, scale=config.logit_scale, cap=0.0)
+    return LayeredCausalModel(config, embed, blocks, norm("final.norm"), head, dtype, embed_norm=norm("embed.norm"))
+
+
 # architecture (lower case) -> builder of its blocks from the checkpoint's tensors
-_BUILDERS = {"dolurax": _build_dolurax, "turutar": _build_turutar, "rezulorn": _build_rezulorn, "sumitar": _build_sumitar}
+_BUILDERS = {"dolurax": _build_dolurax, "turutar": _build_turutar, "rezulorn": _build_rezulorn, "sumitar": _build_sumitar,
+             "vosolorn": _build_vosolorn}
 
 
 def load_layered_model(model_path: str, dtype: str = "bfloat16", config: dict | None = None) -> LayeredCausalModel:

@@ -99,11 +99,11 @@ class StepContext:
         self.cache = cache
         self.buf = model._buffers(self.T)
 
-    def max_keys(self, chunk: int, window: int = 0, keep_first: int = 0) -> int:
+    def max_keys(self, chunk: int, window: int = 0, keep_first: int = 0, pool: int = 0) -> int:
         """The longest key range any tile of the step reads under a chunk size and a window (0: none) that keeps the first
-        `keep_first` positions visible."""
+        `keep_first` positions visible, or one row per block of `pool` positions before it."""
         keys = max(p0 + n - ((p0 // chunk) * chunk if chunk > 0 else 0) for _, n, _, p0 in self._seqs)
-        return min(keys, window + 64 + keep_first) if window > 0 else keys
+        return min(keys, window + 64 + keep_first + (keys // pool if pool > 0 else 0)) if window > 0 else keys
 
     def seqs(self) -> tuple[int, int]:
         """(device pointer, count) of the step's sequences as (first row, rows, slot, first position)"""
@@ -147,14 +147,15 @@ class LayeredCausalModel:
         self._graph_warm: set = set()
         self._gstream: Stream | None = None
         self._tile_sizes = {b.mixer.queries_per_tile for b in blocks if b.mixer.queries_per_tile}
-        self._tops = {b.mlp.spec.top for b in blocks if b.mlp is not None and b.mlp.spec.kind == "moe"}
+        self._tops = {getattr(b.mlp.spec, "slots", b.mlp.spec.top) for b in blocks if b.mlp is not None and b.mlp.spec.kind == "moe"}
 
     # ------------------------------------------------------------------ setup
     def init_cache(self, max_tokens: int = 4096, page_size: int = 64, slots: int = 8) -> PagedKVCache:
         """Allocate the paged cache for about `max_tokens` live positions (it grows when more arrive)."""
         shapes = [self.blocks[li].mixer.spec.cache_shape() for li, _ in self.runs]
         states = [tuple(getattr(self.blocks[li], "state_shapes", ())) for li, _ in self.runs]
-        self.cache = PagedKVCache(shapes, self.dtype, page_size, max_tokens, slots, state_shapes=states)
+        pools = [getattr(self.blocks[li].mixer.spec, "pool", 0) for li, _ in self.runs]
+        self.cache = PagedKVCache(shapes, self.dtype, page_size, max_tokens, slots, state_shapes=states, pools=pools)
         self._graphs.clear()
         self._graph_warm.clear()
         return self.cache

@@ -12,6 +12,10 @@ recurrent mixer, the last inputs of a short convolution): `state[i][j]` is `[slo
 when its slot is handed out again -- the kernels that read it take a sequence whose first position is 0 as starting from
 zero -- and cannot be truncated.
 
+Pooled rows: a layer whose attention sees means of blocks of `pool` positions keeps them beside its pages, in two arrays
+`[pages, kv_heads, rows, dim]` with rows = ceil(page_size / pool): the mean of block b lives with the page that holds the
+block's last position, row b - floor(page_index page_size / pool), so that pages carry their blocks when they change hands.
+
 Growth: when the free list runs dry the pool doubles (device arrays are reallocated and the old pages copied, page
 numbers stay valid); a page table row grows the same way.  Sizing the pool for the expected number of live tokens up
 front (`tokens_hint`) avoids both.
@@ -137,10 +141,12 @@ class PagedKVCache:
     """Device arrays of every layer + the page pool.  `layer_shapes` = [(kv_heads, dim, vdim), ...], one entry per cache
     (a layer that runs several times in a loop has one per run); vdim 0: the layer keeps one array whose rows serve as
     keys and, by a prefix, as values (latent attention) -- `v[i]` is then None; kv_heads 0: the layer has no pages at all.
-    `state_shapes` = per cache the float32 elements per slot of each of its state arrays."""
+    `state_shapes` = per cache the float32 elements per slot of each of its state arrays; `pools` = per cache the block size of
+    its pooled rows (0: none; `pk[i]`, `pv[i]` are then None)."""
 
     def __init__(self, layer_shapes: list[tuple[int, int, int]], dtype: str = "bfloat16", page_size: int = 64,
-                 tokens_hint: int = 4096, slots: int = 8, state_shapes: "list[tuple] | None" = None):
+                 tokens_hint: int = 4096, slots: int = 8, state_shapes: "list[tuple] | None" = None,
+                 pools: "list[int] | None" = None):
         if dtype not in ("bfloat16", "float32"):
             raise ValueError("PagedKVCache: dtype is 'bfloat16' or 'float32'")
         self.dtype = bfloat16 if dtype == "bfloat16" else float32
@@ -150,6 +156,11 @@ class PagedKVCache:
         self.pool = PagePool(page_size, pages, slots, max(4, -(-max(1, tokens_hint) // page_size) + 1))
         self.k: list[GPUArray | None] = []
         self.v: list[GPUArray | None] = []
+        self.pk: list[GPUArray | None] = []
+        self.pv: list[GPUArray | None] = []
+        self.pools = [int(p) for p in (pools or [0] * len(self.layer_shapes))]
+        if len(self.pools) != len(self.layer_shapes) or any(p < 0 for p in self.pools):
+            raise ValueError("PagedKVCache: one block size per cache")
         self._alloc(pages, copy_from=None)
         self.state_shapes = [tuple(int(n) for n in sh) for sh in (state_shapes or [()] * len(self.layer_shapes))]
         if len(self.state_shapes) != len(self.layer_shapes):
@@ -162,22 +173,25 @@ class PagedKVCache:
     def page_size(self) -> int:
         return self.pool.page_size
 
+    def pool_rows(self, i: int) -> int:
+        """rows per page of cache i's pooled arrays"""
+        return -(-self.page_size // self.pools[i]) if self.pools[i] > 0 else 0
+
     def _alloc(self, pages: int, copy_from) -> None:
         ps = self.pool.page_size
-        k_new, v_new = [], []
+        new: list[list] = [[], [], [], []]
         for i, (g, d, dv) in enumerate(self.layer_shapes):
-            k = zeros((pages, g, ps, d), self.dtype) if g > 0 else None
-            v = zeros((pages, g, ps, dv), self.dtype) if dv > 0 and g > 0 else None
-            if copy_from is not None:
-                if k is not None:
-                    api.memcpy_d2d(k.device_ptr, self.k[i].device_ptr, self.k[i].nbytes, _st())
-                if v is not None:
-                    api.memcpy_d2d(v.device_ptr, self.v[i].device_ptr, self.v[i].nbytes, _st())
-            k_new.append(k)
-            v_new.append(v)
+            pr = self.pool_rows(i) if g > 0 and dv > 0 else 0
+            shapes = ((g, ps, d) if g > 0 else None, (g, ps, dv) if dv > 0 and g > 0 else None, (g, pr, d) if pr else None,
+                      (g, pr, dv) if pr else None)
+            for arrays, old, sh in zip(new, (self.k, self.v, self.pk, self.pv), shapes):
+                a = zeros((pages, *sh), self.dtype) if sh is not None else None
+                if copy_from is not None and a is not None:
+                    api.memcpy_d2d(a.device_ptr, old[i].device_ptr, old[i].nbytes, _st())
+                arrays.append(a)
         if copy_from is not None:
             api.device_sync()
-        self.k, self.v = k_new, v_new
+        self.k, self.v, self.pk, self.pv = new
         self._pages_dev = pages
 
     def _alloc_state(self, slots: int, copy_from) -> None:
@@ -227,7 +241,7 @@ class PagedKVCache:
 
     @property
     def nbytes(self) -> int:
-        return (sum(a.nbytes for a in self.k if a is not None) + sum(a.nbytes for a in self.v if a is not None)
+        return (sum(a.nbytes for arrs in (self.k, self.v, self.pk, self.pv) for a in arrs if a is not None)
                 + sum(a.nbytes for arrs in self.state for a in arrs))
 
 

@@ -315,6 +315,8 @@ def random_layered_model(config, dtype: str = "bfloat16", seed: int = 1234, std:
         return _random_pre_norm_model(config, dtype, mat, vec)
     if config.block == "sandwich":
         return _random_sandwich_model(config, dtype, mat, vec)
+    if config.norm == "rmsnorm":
+        return _random_post_rms_model(config, dtype, mat, vec)
     blocks, mixing = [], False
     for i, L in enumerate(config.layers):
         m = L.mixer
@@ -482,3 +484,44 @@ def _random_sandwich_model(config, dtype, mat, vec):
         blocks.append(SandwichBlock(norm(), mixer, norm(), norm2, mlp, norm2b))
     embed = mat(V, W)
     return LayeredCausalModel(config, embed, blocks, norm(), LinearRows(embed), dtype)
+
+
+def _random_post_rms_model(config, dtype, mat, vec):
+    """The RMS-normed post-norm form of `random_layered_model` (windowed attention with pooled blocks, matrix memory with
+    exponential gates, gelu feed-forwards, experts behind a logit router): random matrices, norm weights (with their layer scale)
+    at one, zero router and input-gate biases, forget-gate biases of 3."""
+    from ..core.dtypes import float32
+    from .layers.block import PostNormBlock
+    from .layers.dense_rows import GatedDenseRows
+    from .layers.linear import LinearRows
+    from .layers.matrix_lstm import MatrixLSTMMixer
+    from .layers.moe_rows import GroupedRouterMoE
+    from .layers.norm import RowNorm
+    from .layers.paged_attention import PagedAttentionMixer
+    from .models.layered import LayeredCausalModel
+    W, V, eps = config.hidden_size, config.vocab_size, config.norm_eps
+
+    def norm():
+        return RowNorm("rmsnorm", vec(W, 1.0), None, eps)
+
+    blocks = []
+    for i, L in enumerate(config.layers):
+        m, f = L.mixer, L.mlp
+        proj, o_proj = LinearRows(mat(m.proj_cols, W)), LinearRows(mat(W, m.attn_cols))
+        if m.kind == "attention":
+            mixer = PagedAttentionMixer(m, i, proj, o_proj, vec(m.dim, 1.0), vec(m.dim, 1.0), eps)
+        else:
+            mixer = MatrixLSTMMixer(m, i, proj, o_proj, vec(m.heads, 0.0), vec(m.heads, 3.0), vec(m.heads * m.vdim, 1.0), eps)
+        mlp = None
+        if f is not None and f.kind == "dense":
+            mlp = GatedDenseRows(f, LinearRows(mat(2 * f.ff, W)), LinearRows(mat(W, f.ff)))
+        elif f is not None:
+            n = f.experts + (1 if f.shared_slot else 0)
+            own = bool(f.shared_ff) and not f.shared_slot
+            mlp = GroupedRouterMoE(f, mat(f.experts, W).astype(float32), LinearRows(mat(n, f.ff, W), epilogue=8),
+                                   LinearRows(mat(n, W, f.ff)), LinearRows(mat(f.shared_ff, W), epilogue=8) if own else None,
+                                   LinearRows(mat(W, f.shared_ff)) if own else None, router_bias=vec(f.experts, 0.0))
+        blocks.append(PostNormBlock(mixer, norm(), mlp, norm() if mlp is not None else None, eps))
+    embed = mat(V, W)
+    return LayeredCausalModel(config, embed, blocks, norm(), LinearRows(embed, epilogue=2, scale=config.logit_scale, cap=0.0), dtype,
+                              embed_norm=norm() if config.embed_norm else None)
