@@ -43,6 +43,10 @@ The same for the Rezulorn design of the layered family beside a dense Dolurax st
 The same for the Sumitar design (windowed attention beside a gated linear recurrence, gated delta rule, PolyNorm feed-forward,
 experts with a choice bias) beside a Rezulorn stack at equal sizes, the closest existing model.
 
+    python bench.py --vosolorn [--vosolorn-sizes v-2048,v-4096] [--steps K] [--warmup W]
+The same for the Vosolorn design (the matrix memory of xLSTM, attention with pooled blocks before its window, gelu experts
+behind a logit router) beside a Rezulorn stack at equal sizes, the closest existing model.
+
     python bench.py --turutar [--turutar-sizes t-2048,t-4096] [--steps K] [--warmup W]
 The same for the Turutar design (latent + windowed attention, gated dense feed-forward, token side inputs, a looped pair of
 layers) next to a Dolurax stack of equal size, the closest existing model: same family, same cache and kernels.
@@ -107,6 +111,11 @@ def parse_args():
                          "beside a gated linear recurrence, gated delta rule, mixture of experts with a choice bias) beside a "
                          "Rezulorn stack at equal sizes, one JSON line")
     ap.add_argument("--sumitar-sizes", default="s-2048,s-4096")
+    ap.add_argument("--vosolorn", action="store_true",
+                    help="instead of the default workload: prefill / decode throughput of the Vosolorn design (the matrix memory of "
+                         "xLSTM, attention with pooled blocks before its window, gelu experts behind a logit router) beside a "
+                         "Rezulorn stack at equal sizes, one JSON line")
+    ap.add_argument("--vosolorn-sizes", default="v-2048,v-4096")
     return ap.parse_args()
 
 
@@ -632,6 +641,11 @@ def run_ours(args) -> None:
 
 def main():
     args = parse_args()
+    if args.vosolorn:
+        sys.path.insert(0, os.path.join(ROOT, "scripts"))
+        import bench_layered
+        print(json.dumps(bench_layered.main_vosolorn(ROOT, args.vosolorn_sizes.split(","), args.steps, args.warmup)))
+        return
     if args.sumitar:
         sys.path.insert(0, os.path.join(ROOT, "scripts"))
         import bench_layered

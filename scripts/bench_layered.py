@@ -61,6 +61,16 @@ SUMITAR_SIZES = {
 }
 
 
+# Vosolorn: post-norm blocks; two matrix-memory layers (a gated dense feed-forward; experts without gates and a shared one, whose
+# chosen matrices together have the dense size) and an attention layer with a window and pooled blocks before it
+VOSOLORN_SIZES = {
+    "v-2048": dict(width=2048, heads=16, kv_heads=4, dim=128, window=1024, pool=16, rot=64, lin_heads=16, lin_dim=128, lin_vdim=128,
+                   ff=8192, experts=16, top=3, eff=2048, shared_ff=2048, vocab=32768),
+    "v-4096": dict(width=4096, heads=32, kv_heads=8, dim=128, window=2048, pool=16, rot=64, lin_heads=8, lin_dim=256, lin_vdim=512,
+                   ff=12288, experts=16, top=3, eff=3072, shared_ff=3072, vocab=32768),
+}
+
+
 def peaks(root: str) -> tuple[float, float, str]:
     p = os.path.join(root, "MEASURED_PEAKS.json")
     if os.path.exists(p):
@@ -232,6 +242,70 @@ def sumitar_twin_bytes_flops(s: dict, T: int, B: int, ctx: int) -> tuple[float, 
     state = 2 * 4 * Hl * Dl * Dvl
     dec = 2 * weights + B * (2 * 2 * G * D * ctx + 2 * state) + 2 * s["vocab"] * W
     attn_fl = 2 * T * H * (T / 2) * 2 * D + 2 * 2 * T * Hl * 4 * Dl * Dvl
+    return float(dec), float(2 * T * weights + attn_fl + 2 * s["vocab"] * W)
+
+
+def vosolorn_config(s: dict):
+    from pygpukit_b200.llm.config import layered_config_from_json
+    dense = {"kind": "dense", "ff": s["ff"]}
+    moe = {"kind": "moe", "expert": {"ff": s["eff"]}, "router": {"experts": s["experts"], "top": s["top"]}, "shared": {"ff": s["shared_ff"]}}
+    memory = {"heads": s["lin_heads"], "dim": s["lin_dim"], "vdim": s["lin_vdim"], "gate_cap": 15.0}
+    attention = {"heads": s["heads"], "kv_heads": s["kv_heads"], "dim": s["dim"], "vdim": s["dim"], "scale": s["dim"] ** -0.5,
+                 "mask": {"size": s["window"], "pool": s["pool"]}, "rot": {"dims": s["rot"], "base": 10000.0}}
+    layers = [{"type": "mlstm", "mlp": dense, "mixer": memory}, {"type": "mlstm", "mlp": moe, "mixer": memory},
+              {"type": "attention", "mlp": dense, "mixer": attention}]
+    return layered_config_from_json({"architecture": "Vosolorn", "layers": layers, "norm": {"eps": 1e-6}, "logit_scale": 1.0,
+                                     "vocab": s["vocab"], "width": s["width"]})
+
+
+def vosolorn_twin_config(s: dict):
+    """The closest existing model at equal size: a Rezulorn stack of two lightning layers (decayed linear attention with
+    per-sequence state) and a windowed attention layer, the same heads, squared-ReLU feed-forward of the dense size (two matrices to
+    the gated form's three) in all of them."""
+    from pygpukit_b200.llm.config import layered_config_from_json
+    mlp = {"kind": "dense", "ff": s["ff"]}
+    H, G, D, Hl, Dl, Dvl = s["heads"], s["kv_heads"], s["dim"], s["lin_heads"], s["lin_dim"], s["lin_vdim"]
+    decay = [1.0 - 2.0 ** (-5.0 - 5.0 * h / max(1, Hl - 1)) for h in range(Hl)]
+    lightning = {"type": "lightning", "mlp": mlp, "mixer": {"heads": Hl, "dim": Dl, "vdim": Dvl, "decay": decay}}
+    attention = {"type": "attention", "mlp": mlp, "mixer": {"heads": H, "kv_heads": G, "dim": D, "vdim": D, "scale": D ** -0.5,
+                                                             "mask": {"size": s["window"], "keep_first": 4}}}
+    return layered_config_from_json({"architecture": "Rezulorn", "layers": [lightning, lightning, attention], "canon": {"taps": 4},
+                                     "norm": {"eps": 1e-6}, "residual_mult": 0.5, "logit_scale": 1.0, "vocab": s["vocab"], "width": s["width"]})
+
+
+def _vosolorn_parts(s: dict, T: int, ctx: int) -> tuple[float, float, float, float, float]:
+    """(matrix-memory weights, attention weights, keys a decoded token sees, mean keys a prompt's token sees, state bytes)"""
+    W, H, G, D = s["width"], s["heads"], s["kv_heads"], s["dim"]
+    Hl, Dl, Dvl, win = s["lin_heads"], s["lin_dim"], s["lin_vdim"], s["window"]
+    mem_w = (2 * Hl * Dl + 2 * Hl * Dvl) * W + W * Hl * Dvl
+    att_w = (H * D + 2 * G * D) * W + W * H * D
+    seen_avg = T / 2 if T <= win else win * (1 - win / (2 * T))
+    return mem_w, att_w, min(ctx, win), seen_avg, 2 * 4 * Hl * Dl * Dvl
+
+
+def vosolorn_bytes_flops(s: dict, T: int, B: int, ctx: int) -> tuple[float, float]:
+    """(bytes a decode step of B tokens touches, FLOPs of a T-token prefill; the matrix memory counted in its recurrent form)"""
+    W, H, G, D, win, pool = s["width"], s["heads"], s["kv_heads"], s["dim"], s["window"], s["pool"]
+    Hl, Dl, Dvl = s["lin_heads"], s["lin_dim"], s["lin_vdim"]
+    mem_w, att_w, seen, seen_avg, state = _vosolorn_parts(s, T, ctx)
+    mem_w += 2 * Hl * W
+    seen += max(0, ctx - win) // pool
+    seen_avg += max(0, T - win) ** 2 / (2 * T * pool)
+    dense_w = 3 * s["ff"] * W
+    act = min(s["experts"], B * s["top"])
+    moe_w = s["experts"] * W * 2 + 2 * s["shared_ff"] * W + act * 2 * s["eff"] * W          # the router is float32
+    dec = 2 * (2 * mem_w + att_w + 2 * dense_w + moe_w) + B * (2 * 2 * G * D * seen + 2 * state) + 2 * s["vocab"] * W
+    per_tok = 2 * mem_w + att_w + 2 * dense_w + s["experts"] * W + 2 * s["shared_ff"] * W + s["top"] * 2 * s["eff"] * W
+    attn_fl = 2 * T * H * seen_avg * 2 * D + 2 * T * Hl * 4 * Dl * Dvl
+    return float(dec), float(2 * T * per_tok + attn_fl + 2 * s["vocab"] * W)
+
+
+def vosolorn_twin_bytes_flops(s: dict, T: int, B: int, ctx: int) -> tuple[float, float]:
+    W, H, G, D = s["width"], s["heads"], s["kv_heads"], s["dim"]
+    mem_w, att_w, seen, seen_avg, state = _vosolorn_parts(s, T, ctx)
+    weights = 2 * mem_w + att_w + 3 * 2 * s["ff"] * W
+    dec = 2 * weights + B * (2 * 2 * G * D * seen + 2 * state) + 2 * s["vocab"] * W
+    attn_fl = 2 * T * H * seen_avg * 2 * D + 2 * T * s["lin_heads"] * 4 * s["lin_dim"] * s["lin_vdim"]
     return float(dec), float(2 * T * weights + attn_fl + 2 * s["vocab"] * W)
 
 
@@ -423,6 +497,27 @@ def main_sumitar(root: str, sizes: list[str], steps: int, warm: int, prompt: int
                                        (1, 8), steps, max(3, warm), hbm, tflops)
         api.device_sync()
         entry["rezulorn_twin"] = run_layered(sumitar_twin_config(s), lambda T, B, ctx: sumitar_twin_bytes_flops(s, T, B, ctx), s["vocab"],
+                                             prompt, (1, 8), steps, max(3, warm), hbm, tflops)
+        api.device_sync()
+        res["sizes"][name] = entry
+    return res
+
+
+def main_vosolorn(root: str, sizes: list[str], steps: int, warm: int, prompt: int = 2000) -> dict:
+    """Vosolorn beside a Rezulorn stack of the same family at equal size (two state-only layers and a windowed attention layer):
+    prefill of `prompt` tokens, decode of 1 and 8 requests at that context."""
+    from pygpukit_b200._lib import api
+    hbm, tflops, src = peaks(root)
+    res = {"metric": "vosolorn_prefill_decode_tokens_per_s", "data": "synthetic",
+           "dtype": "bf16 matrices and cache, f32 residual / norms / scores / router / gates / recurrent state",
+           "peaks": {"hbm_gbs": hbm, "bf16_tflops": tflops, "source": src}, "prompt": prompt, "steps": steps, "warmup": warm, "sizes": {}}
+    for name in sizes:
+        s = VOSOLORN_SIZES[name]
+        entry = {"shape": dict(s)}
+        entry["vosolorn"] = run_layered(vosolorn_config(s), lambda T, B, ctx: vosolorn_bytes_flops(s, T, B, ctx), s["vocab"], prompt,
+                                        (1, 8), steps, max(3, warm), hbm, tflops)
+        api.device_sync()
+        entry["rezulorn_twin"] = run_layered(vosolorn_twin_config(s), lambda T, B, ctx: vosolorn_twin_bytes_flops(s, T, B, ctx), s["vocab"],
                                              prompt, (1, 8), steps, max(3, warm), hbm, tflops)
         api.device_sync()
         res["sizes"][name] = entry
