@@ -106,10 +106,18 @@ __device__ __forceinline__ void pool_block_rows(const PrepRotArgs& a, int pos, i
     const TC* src = (const TC*)(is_v ? a.vc : a.kc);
     TC* dst = (TC*)(is_v ? a.pv : a.pk) + (((size_t)tab[lastpg] * a.G + g) * a.pool_rows + row) * n;
     const float inv = 1.f / (float)P;
-    for (int d = lane; d < n; d += 32) {
-        float s = 0.f;
-        for (int j = pos - P; j < pos; ++j) s += cload<TC>(src + (((size_t)tab[j / a.PS] * a.G + g) * a.PS + j % a.PS) * n + d);
-        cstore<TC>(dst + d, s * inv);
+    for (int d0 = lane; d0 < n; d0 += 128) {           // four elements per lane and several rows in flight
+        float s[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll 4
+        for (int j = pos - P; j < pos; ++j) {
+            const TC* r = src + (((size_t)tab[j / a.PS] * a.G + g) * a.PS + j % a.PS) * n;
+#pragma unroll
+            for (int e = 0; e < 4; ++e)
+                if (d0 + 32 * e < n) s[e] += cload<TC>(r + d0 + 32 * e);
+        }
+#pragma unroll
+        for (int e = 0; e < 4; ++e)
+            if (d0 + 32 * e < n) cstore<TC>(dst + d0 + 32 * e, s[e] * inv);
     }
 }
 
@@ -298,9 +306,10 @@ __device__ __forceinline__ int blocks_seen(const AttnArgs& a, int pos) {
     const int past = pos - a.window + 1;                 // positions below `past` have left the window
     return past > 0 ? past / a.pool : 0;
 }
-__device__ __forceinline__ int early_rows(const AttnArgs& a, int jlo, int jhi) {
+// EXT: the kernels' form that knows pooled blocks and outputs turned back (the other designs run the form without)
+template <bool EXT> __device__ __forceinline__ int early_rows(const AttnArgs& a, int jlo, int jhi) {
     if (a.window <= 0) return 0;
-    return a.pool > 0 ? blocks_seen(a, jhi) : min(a.keep, jlo);
+    return EXT && a.pool > 0 ? blocks_seen(a, jhi) : min(a.keep, jlo);
 }
 // element offset of pooled block b of KV head g, before the factor of the row size
 __device__ __forceinline__ long long pooled_row(const AttnArgs& a, int slot, int g, int b) {
@@ -358,7 +367,7 @@ __device__ __forceinline__ void stage_rows(float* dst, int ld, const TC* base, c
 constexpr int PPW = 4;                  // (query, head) pairs per warp
 constexpr int NWARP = 8;
 
-template <typename TC, int NV>
+template <typename TC, int NV, bool EXT>
 __global__ void __launch_bounds__(256) seq_attention_kernel(AttnArgs a) {
     extern __shared__ __align__(16) float sm[];
     const int D = a.D, Dv = a.Dv, DP = D + 1;
@@ -415,13 +424,13 @@ __global__ void __launch_bounds__(256) seq_attention_kernel(AttnArgs a) {
     const TC* kc = (const TC*)a.kc;
     const TC* vc = (const TC*)a.vc;
     // this block's slice of the key tiles (all of them when splits == 1)
-    const int kept = early_rows(a, jlo, jhi), nkept = (kept + KT - 1) / KT;
+    const int kept = early_rows<EXT>(a, jlo, jhi), nkept = (kept + KT - 1) / KT;
     const int ntile = nkept + (jhi - jlo) / KT + 1, per = (ntile + a.splits - 1) / a.splits;
     const int tbeg = (int)blockIdx.z * per, tend = min(ntile, tbeg + per);
     for (int ti = tbeg; ti < tend; ++ti) {
         const int j0 = ti < nkept ? ti * KT : jlo + (ti - nkept) * KT;
         const int jmax = ti < nkept ? kept - 1 : jhi;
-        const bool pooled = a.pool > 0 && ti < nkept;
+        const bool pooled = EXT && a.pool > 0 && ti < nkept;
         __syncthreads();
         if (threadIdx.x < KT) {
             const int j = j0 + threadIdx.x;
@@ -543,7 +552,7 @@ __global__ void __launch_bounds__(256) seq_attention_kernel(AttnArgs a) {
             float o = 0.f;
 #pragma unroll 8
             for (int sp = 0; sp < a.splits; ++sp) o = fmaf(wsl[p][sp], __ldcg(rec + (size_t)sp * (Dv + 2)), o);
-            if (a.o_inv_freq) {
+            if (EXT && a.o_inv_freq) {
                 const float* rp = rec - dv + turn_partner(a, dv);
                 float op = 0.f;
 #pragma unroll 8
@@ -555,7 +564,7 @@ __global__ void __launch_bounds__(256) seq_attention_kernel(AttnArgs a) {
         }
         return;
     }
-    if (a.o_inv_freq) {                                // a pair's elements meet through shared memory (the query tile is done)
+    if (EXT && a.o_inv_freq) {                         // a pair's elements meet through shared memory (the query tile is done)
         float* ob = qs + warp * D * PPW;               // [D * PPW] floats of this warp; rows longer than that go through K's tile
         const bool fits = Dv <= D * PPW;
         if (!fits) { __syncthreads(); ob = Ks + warp * Dv; }
@@ -587,8 +596,8 @@ __global__ void __launch_bounds__(256) seq_attention_kernel(AttnArgs a) {
     }
 }
 
-template <typename TC, int NV>
-int launch_attn(const AttnArgs& a, int tiles, cudaStream_t st) {
+template <typename TC, int NV, bool EXT>
+int launch_attn_form(const AttnArgs& a, int tiles, cudaStream_t st) {
     size_t smem = sizeof(float) * ((size_t)NWARP * a.D * PPW + (size_t)KT * (a.D + 1) + (a.valias ? 0 : (size_t)KT * a.Dv));
     if (a.o_inv_freq) {                     // turning the outputs back needs a value row per warp behind the queries
         const size_t turn = sizeof(float) * ((size_t)NWARP * a.D * PPW + (size_t)NWARP * a.Dv);
@@ -598,12 +607,19 @@ int launch_attn(const AttnArgs& a, int tiles, cudaStream_t st) {
     static size_t configured = 0;
     // the opt-in is needed once dynamic + STATIC shared memory (row offsets, the fold's slice weights: ~9 KB) pass 48 KB
     if (smem > 32 * 1024 && configured == 0) {
-        PGK_CUDA(cudaFuncSetAttribute(seq_attention_kernel<TC, NV>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
+        PGK_CUDA(cudaFuncSetAttribute(seq_attention_kernel<TC, NV, EXT>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
         configured = 1;
     }
     const int rep = a.H / a.G, hsplit = (rep + a.HB - 1) / a.HB;
-    PGK_CUDA(launch(seq_attention_kernel<TC, NV>, dim3(tiles, a.G * hsplit, a.splits), dim3(256), smem, st, a));
+    PGK_CUDA(launch(seq_attention_kernel<TC, NV, EXT>, dim3(tiles, a.G * hsplit, a.splits), dim3(256), smem, st, a));
     return 0;
+}
+
+inline bool extended(const AttnArgs& a) { return a.pool > 0 || a.o_inv_freq; }
+
+template <typename TC, int NV>
+int launch_attn(const AttnArgs& a, int tiles, cudaStream_t st) {
+    return extended(a) ? launch_attn_form<TC, NV, true>(a, tiles, st) : launch_attn_form<TC, NV, false>(a, tiles, st);
 }
 
 template <typename TC>
@@ -668,7 +684,7 @@ __device__ __forceinline__ void load_values(const TC* p, bool vec, int n_left, f
     for (int i = 0; i < NV; ++i) out[i] = i < n_left ? cload<TC>(p + i) : 0.f;
 }
 
-template <typename TC, int NV, int DPAIRS>
+template <typename TC, int NV, int DPAIRS, bool EXT>
 __global__ void __launch_bounds__(256) seq_attention_decode_kernel(AttnArgs a) {
     extern __shared__ __align__(16) float sm[];
     const int D = a.D, Dv = a.Dv;
@@ -706,7 +722,7 @@ __global__ void __launch_bounds__(256) seq_attention_decode_kernel(AttnArgs a) {
     }
     // ... and the page of the warp's first key tile
     const int jlo = first_key(a, pos), jhi = pos;
-    const int kept = early_rows(a, jlo, jhi), nkept = (kept + KT - 1) / KT;
+    const int kept = early_rows<EXT>(a, jlo, jhi), nkept = (kept + KT - 1) / KT;
     const int ntile = nkept + (jhi - jlo) / KT + 1, per = (ntile + a.splits - 1) / a.splits;
     const int tb = (int)blockIdx.z * per, te = min(ntile, tb + per);
     int page_first = 0;
@@ -714,7 +730,7 @@ __global__ void __launch_bounds__(256) seq_attention_decode_kernel(AttnArgs a) {
         const int ti = tb + warp;
         const bool early = ti < nkept;
         const int j = (early ? ti * KT : jlo + (ti - nkept) * KT) + lane;
-        const int at = a.pool > 0 && early ? j * a.pool + a.pool - 1 : j;          // a pooled block: its last position
+        const int at = EXT && a.pool > 0 && early ? j * a.pool + a.pool - 1 : j;          // a pooled block: its last position
         if (ti < te && j <= (early ? kept - 1 : jhi)) page_first = a.table[(size_t)slot * a.max_pages + at / a.PS];
     }
     __syncthreads();
@@ -735,7 +751,7 @@ __global__ void __launch_bounds__(256) seq_attention_decode_kernel(AttnArgs a) {
     for (int ti = tb + warp; ti < te; ti += NWARP) {
         const int j0 = ti < nkept ? ti * KT : jlo + (ti - nkept) * KT, jmax = ti < nkept ? kept - 1 : jhi;
         const int j = j0 + lane;
-        const bool in = j <= jmax, pooled = a.pool > 0 && ti < nkept;
+        const bool in = j <= jmax, pooled = EXT && a.pool > 0 && ti < nkept;
         const TC* kc = (const TC*)(pooled ? a.pk : a.kc);
         const TC* vc = (const TC*)(pooled ? a.pv : a.vc);
         long long ko = 0, vo = 0;
@@ -842,7 +858,7 @@ __global__ void __launch_bounds__(256) seq_attention_decode_kernel(AttnArgs a) {
     }
     __syncthreads();
     const size_t t = t0;
-    const bool turn = a.o_inv_freq && a.splits == 1;
+    const bool turn = EXT && a.o_inv_freq && a.splits == 1;
     for (int i = threadIdx.x; i < nh * Dv; i += blockDim.x) {
         const int p = i / Dv, dv = i - p * Dv, dp = turn ? turn_partner(a, dv) : dv;
         float M = -INFINITY;
@@ -920,7 +936,7 @@ __global__ void __launch_bounds__(256) seq_attention_decode_kernel(AttnArgs a) {
         float o = 0.f;
 #pragma unroll 8
         for (int sp = 0; sp < a.splits; ++sp) o = fmaf(wsl[p][sp], __ldcg(rec + (size_t)sp * (Dv + 2)), o);
-        if (a.o_inv_freq) {
+        if (EXT && a.o_inv_freq) {
             const float* rp = rec - dv + turn_partner(a, dv);
             float op = 0.f;
 #pragma unroll 8
@@ -940,18 +956,23 @@ __global__ void __launch_bounds__(256) seq_attention_decode_kernel(AttnArgs a) {
     }
 }
 
-template <typename TC, int NV, int DPAIRS>
-int launch_attn_decode_dp(const AttnArgs& a, int tiles, cudaStream_t st) {
+template <typename TC, int NV, int DPAIRS, bool EXT>
+int launch_attn_decode_form(const AttnArgs& a, int tiles, cudaStream_t st) {
     const size_t smem = sizeof(float) * ((size_t)DPAIRS * a.D + 2 * NWARP * DPAIRS + (size_t)NWARP * DPAIRS * a.Dv);
     PGK_REQUIRE(smem <= 200 * 1024, "seq_attention failed: head sizes %d / %d need %zu bytes of shared memory", a.D, a.Dv, smem);
     static bool configured = false;
     if (smem > 32 * 1024 && !configured) {            // dynamic + static shared memory may pass 48 KB from here on
-        PGK_CUDA(cudaFuncSetAttribute(seq_attention_decode_kernel<TC, NV, DPAIRS>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
+        PGK_CUDA(cudaFuncSetAttribute(seq_attention_decode_kernel<TC, NV, DPAIRS, EXT>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
         configured = true;
     }
     const int rep = a.H / a.G, hsplit = (rep + DPAIRS - 1) / DPAIRS;
-    PGK_CUDA(launch(seq_attention_decode_kernel<TC, NV, DPAIRS>, dim3(tiles, a.G * hsplit, a.splits), dim3(256), smem, st, a));
+    PGK_CUDA(launch(seq_attention_decode_kernel<TC, NV, DPAIRS, EXT>, dim3(tiles, a.G * hsplit, a.splits), dim3(256), smem, st, a));
     return 0;
+}
+
+template <typename TC, int NV, int DPAIRS>
+int launch_attn_decode_dp(const AttnArgs& a, int tiles, cudaStream_t st) {
+    return extended(a) ? launch_attn_decode_form<TC, NV, DPAIRS, true>(a, tiles, st) : launch_attn_decode_form<TC, NV, DPAIRS, false>(a, tiles, st);
 }
 
 // Few blocks (one or a handful of requests): two heads per block instead of eight -- four times the blocks, a quarter of

@@ -14,7 +14,7 @@
 //              memory, and block 0 writes n and m once all blocks have read them.
 //   prompts    chunks of 64 tokens, all at once.  With F the running sum of f inside a chunk,
 //              m_t = max(F_t + m_in, max_(s<=t) (F_t - F_s + i_s)) for every t, so that
-//              1. gates:   F, i, m of every token (a warp per sequence and head: one scan of (sum, maximum) pairs);
+//              1. gates:   F, i, m of every token (a block per sequence and head: one scan of (sum, maximum) pairs);
 //              2. update:  U_c = sum_s e^(F_end - F_s + i_s - m_end) k_s v_s^T per chunk (and the n part);
 //              3. scan:    per state element over the chunks in order, leaving the state BEFORE each chunk in the workspace;
 //              4. output:  o_t = e^(F_t + m_in - m_t) S_c^T q_t + sum_(s<=t) e^(F_t - F_s + i_s - m_t) (q_t.k_s) v_s over the
@@ -193,24 +193,28 @@ struct GateWs {                          // per (row, head), row-major [T][H]
     float* gi; float* m; float* mp;      // i, m, and m before the token
 };
 
-__global__ void __launch_bounds__(128) mlstm_gates_kernel(MlstmArgs a, GateWs g) {
-    const int lane = threadIdx.x & 31, h = blockIdx.y * 4 + (threadIdx.x >> 5);
-    if (h >= a.H) return;
+constexpr int GT = 256;                  // tokens per round of the gate scan, one per thread
+
+// A block per (sequence, head): every round takes GT tokens, scans (sum of f, running maximum) pairs inside the warps, then over the
+// warps' totals.  (F1, m1) then (F2, m2) compose to (F1 + F2, max(m1 + F2, m2)).
+__global__ void __launch_bounds__(GT) mlstm_gates_kernel(MlstmArgs a, GateWs g) {
+    __shared__ double wF[GT / 32], wm[GT / 32], Fat[GT / MC], last_m;
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, h = blockIdx.y;
     const int4 sq = a.seqs[blockIdx.x];
     float* Mrow = a.M + (size_t)sq.z * a.H + h;
-    double m_in = sq.w > 0 ? (double)*Mrow : 0.0, Fc = 0.0;
+    double m_in = sq.w > 0 ? (double)*Mrow : 0.0;
     const float ib = a.ib[h], fb = a.fb[h];
     float zi = 0.f, zf = 0.f;
-    if (lane < sq.y) {
-        const float* row = a.proj + (size_t)(sq.x + lane) * a.ld;
+    if (tid < sq.y) {
+        const float* row = a.proj + (size_t)(sq.x + tid) * a.ld;
         zi = row[a.i_off + h]; zf = row[a.f_off + h];
     }
-    for (int t0 = 0; t0 < sq.y; t0 += 32) {
-        const int t = t0 + lane;
+    for (int t0 = 0; t0 < sq.y; t0 += GT) {
+        const int t = t0 + tid;
         const bool in = t < sq.y;
         const float li = log_in(zi + ib, a.cap), lf = log_forget(zf + fb, a.cap);
-        if (t + 32 < sq.y) {                               // the next group's logits travel meanwhile
-            const float* row = a.proj + (size_t)(sq.x + t + 32) * a.ld;
+        if (t + GT < sq.y) {                               // the next round's logits travel meanwhile
+            const float* row = a.proj + (size_t)(sq.x + t + GT) * a.ld;
             zi = row[a.i_off + h]; zf = row[a.f_off + h];
         }
         double F = in ? (double)lf : 0.0, mx = in ? (double)li : -1e300;
@@ -219,18 +223,24 @@ __global__ void __launch_bounds__(128) mlstm_gates_kernel(MlstmArgs a, GateWs g)
             const double Fp = __shfl_up_sync(0xffffffffu, F, o), mxp = __shfl_up_sync(0xffffffffu, mx, o);
             if (lane >= o) { mx = fmax(mx, mxp + F); F += Fp; }
         }
-        const double m = fmax(F + m_in, mx);
+        __syncthreads();                                   // the round before has read the shared arrays
+        if (lane == 31) { wF[warp] = F; wm[warp] = mx; }
+        __syncthreads();
+        double Fw = 0.0, mw = m_in;                        // F and m before this warp's tokens
+        for (int w = 0; w < warp; ++w) { mw = fmax(mw + wF[w], wm[w]); Fw += wF[w]; }
+        const double m = fmax(F + mw, mx);
         double mp = __shfl_up_sync(0xffffffffu, m, 1);
-        if (lane == 0) mp = m_in;
-        if (t0 % MC == 0) Fc = 0.0;
+        if (lane == 0) mp = mw;
+        if (tid % MC == 0) Fat[tid / MC] = Fw;             // the sum in front of every chunk of the round
+        if (t == min(sq.y, t0 + GT) - 1) last_m = m;
+        __syncthreads();
         if (in) {
             const size_t at = (size_t)(sq.x + t) * a.H + h;
-            g.F[at] = Fc + F; g.gi[at] = li; g.m[at] = (float)m; g.mp[at] = (float)mp;
+            g.F[at] = Fw - Fat[tid / MC] + F; g.gi[at] = li; g.m[at] = (float)m; g.mp[at] = (float)mp;
         }
-        Fc += __shfl_sync(0xffffffffu, F, 31);
-        m_in = __shfl_sync(0xffffffffu, m, min(31, sq.y - 1 - t0));
+        m_in = last_m;
     }
-    if (lane == 0) *Mrow = (float)m_in;
+    if (tid == 0) *Mrow = (float)m_in;
 }
 
 // ---------------------------------------------------------------- prompts: chunk update
@@ -374,10 +384,19 @@ constexpr int SLAB = 16;                 // state rows per slab
 __device__ __forceinline__ void stage_transposed(const float* src, int ld, int nc, int D, float mult, float* dst) {
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, dl = lane & 7, tl = lane >> 3;
     const int nd = (D + 7) / 8;
-#pragma unroll 4
-    for (int u = warp; u < nd * (MC / 4); u += 8) {
-        const int d = (u % nd) * 8 + dl, t = (u / nd) * 4 + tl;
-        if (d < D) dst[d * MP + t] = t < nc ? src[(size_t)t * ld + d] * mult : 0.f;
+    constexpr int B = 8;                                   // loads in flight per thread
+    for (int u0 = warp; u0 < nd * (MC / 4); u0 += 8 * B) {
+        float r[B];
+#pragma unroll
+        for (int b = 0; b < B; ++b) {
+            const int u = u0 + 8 * b, d = (u % nd) * 8 + dl, t = (u / nd) * 4 + tl;
+            r[b] = (d < D && t < nc) ? __ldg(src + (size_t)t * ld + d) : 0.f;
+        }
+#pragma unroll
+        for (int b = 0; b < B; ++b) {
+            const int u = u0 + 8 * b, d = (u % nd) * 8 + dl, t = (u / nd) * 4 + tl;
+            if (d < D && t < MC) dst[d * MP + t] = r[b] * mult;
+        }
     }
 }
 
@@ -392,8 +411,10 @@ __global__ void __launch_bounds__(256, 2) mlstm_output_kernel(ChunkArgs p) {
     float* R1 = Qt + D * MP;             // K transposed [D][MP], then V [MC][cw], then the outputs [MC][cw]
     float* At = R1 + r1;                 // [MC][MP]: weight of key s for query t at [s][t]
     float* slab = At + MC * MP;          // [2][SLAB][cw]
-    __shared__ double Fs[MC];
-    __shared__ float is[MC], ms[MC], win[MC], den[MC];
+    // the exponent F_t - F_s + i_s - m_t = (F_t - m_t) + (i_s - F_s), either part as a pair of floats: the sum of the leading parts
+    // is rounded relative to the exponent itself, however large F has grown
+    __shared__ float2 rt[MC], cs[MC];
+    __shared__ float ms[MC], win[MC], den[MC];
     const int4 sq = a.seqs[blockIdx.y];
     const int c = p.c_begin + blockIdx.x, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     if (c * MC >= sq.y || nv <= 0) return;
@@ -428,7 +449,10 @@ __global__ void __launch_bounds__(256, 2) mlstm_output_kernel(ChunkArgs p) {
         const size_t at = (size_t)(r0 + min(tid, nc - 1)) * a.H + h;
         const double F = p.g.F[at];
         const float m = p.g.m[at];
-        Fs[tid] = F; is[tid] = p.g.gi[at]; ms[tid] = m;
+        const double r = F - (double)m, c0 = (double)p.g.gi[at] - F;
+        rt[tid] = make_float2((float)r, (float)(r - (double)(float)r));
+        cs[tid] = make_float2((float)c0, (float)(c0 - (double)(float)c0));
+        ms[tid] = m;
         win[tid] = has_state ? expf((float)(F + (double)p.g.mp[(size_t)r0 * a.H + h] - (double)m)) : 0.f;
     }
     __syncthreads();
@@ -445,15 +469,17 @@ __global__ void __launch_bounds__(256, 2) mlstm_output_kernel(ChunkArgs p) {
 #pragma unroll
                     for (int j = 0; j < 4; ++j) acc[i][j] = fmaf(qq[i], kk[j], acc[i][j]);
             }
+#pragma unroll
+            for (int j = 0; j < 4; ++j)
+#pragma unroll
+                for (int i = 0; i < 4; ++i) {
+                    const float2 r = rt[t0 + i], c2 = cs[s0 + j];
+                    acc[i][j] = (s0 + j <= t0 + i && t0 + i < nc) ? acc[i][j] * expf((r.x + c2.x) + (r.y + c2.y)) : 0.f;
+                }
         }
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
-            float r[4];
-#pragma unroll
-            for (int i = 0; i < 4; ++i) {
-                const int t = t0 + i, s = s0 + j;
-                r[i] = (s <= t && t < nc) ? acc[i][j] * expf((float)(Fs[t] - Fs[s] + (double)is[s] - (double)ms[t])) : 0.f;
-            }
+            const float r[4] = {acc[0][j], acc[1][j], acc[2][j], acc[3][j]};
             *(float4*)(At + (s0 + j) * MP + t0) = make_float4(r[0], r[1], r[2], r[3]);
         }
     }
@@ -464,8 +490,10 @@ __global__ void __launch_bounds__(256, 2) mlstm_output_kernel(ChunkArgs p) {
         const int t = tid >> 2, q = tid & 3;
         const float* Nc = Sc + (size_t)D * Dv;
         float x = 0.f, y = 0.f;
+#pragma unroll 4
         for (int s = q; s <= t; s += 4) x += At[s * MP + t];
         if (has_state)
+#pragma unroll 8
             for (int d = q; d < D; d += 4) y = fmaf(Qt[d * MP + t], __ldg(Nc + d), y);
         x = fmaf(y, win[t], x);
         x += __shfl_xor_sync(0xffffffffu, x, 1);
@@ -617,7 +645,7 @@ int pgk_seq_mlstm_gates(const float* proj, int ld, int i_off, int f_off, const f
     a.seqs = (const int4*)seqs; a.H = heads;
     const size_t n = (size_t)tokens * heads;
     GateWs g{(double*)gates, gates + 2 * n, gates + 3 * n, gates + 4 * n};
-    PGK_CUDA(launch(mlstm_gates_kernel, dim3(n_seqs, (heads + 3) / 4), dim3(128), 0, (cudaStream_t)stream, a, g));
+    PGK_CUDA(launch(mlstm_gates_kernel, dim3(n_seqs, heads), dim3(GT), 0, (cudaStream_t)stream, a, g));
     return 0;
 }
 
