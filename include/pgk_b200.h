@@ -624,6 +624,12 @@ int pgk_rms_pair_rows_f32(const float* a, const float* weight_a, const float* b,
 int pgk_polynorm_rows_f32(float* z, int ld, const float* coef, float eps, int rows, int n, void* stream);
 int pgk_moe_route_biased(const float* logits, int ld, int tokens, int outputs, int real_experts, int top, const float* bias,
                          int renorm, int32_t* idx, int32_t* mat, float* weights, int32_t* rank, int32_t* counts, void* stream);
+/* Router with sigmoid scores: chosen by score + bias among the members of the group_keep best of group_count groups (ranked by the
+ * sum of their two largest choice scores), weights scale * score.  extra >= 0: every token also takes that matrix as its last slot
+ * with weight sigmoid(logits[t, experts]). */
+int pgk_moe_route_sigmoid(const float* logits, int ld, int tokens, int experts, int top, const float* bias, int group_count,
+                          int group_keep, float scale, int extra, int32_t* idx, float* weights, int32_t* rank, int32_t* counts,
+                          void* stream);
 int pgk_moe_combine_rows_f32(const float* parts, const int32_t* inv, const int32_t* mat, const float* weights, int top,
                              const float* self_rows, const float* shared_rows, const float* gate_rows, int ldg, int gate_off,
                              float* out, int rows, int width, void* stream);
@@ -693,6 +699,23 @@ int pgk_seq_mlstm_chunks(const float* proj, int ld, int q_off, int k_off, int v_
                          const float* gates, int chunk_begin, int chunks, float* workspace, void* stream);
 int pgk_seq_mlstm_fused_finish(int vdim);
 
+/* Gated linear attention with a decay per head, token and key channel (seq_gla.cu) on rows that hold q, k [heads x dim], v, gate
+ * [heads x vdim] and `inner` columns y: a = sigmoid(w2^T y + b2)^inv_tau with w2 [inner][heads x dim], S <- diag(a) S + k v^T,
+ * o = q_scale S^T q / its root mean square * weight * silu(gate).  S: [slots][heads][dim][vdim].
+ * _step: one token per sequence, one launch.  Longer steps: _decays once (L: [tokens][heads x dim] floats), then _chunks over
+ * segments of chunks of pgk_seq_gla_chunk_tokens tokens (0: keys too large; workspace: n_seqs x chunks x heads x dim (vdim + 1)
+ * floats).  With pgk_seq_gla_fused_finish(vdim) == 0 the chunks leave plain outputs and pgk_seq_linear_finish is to follow. */
+int pgk_seq_gla_chunk_tokens(int dim, int vdim);
+int pgk_seq_gla_fused_finish(int vdim);
+int pgk_seq_gla_step(const float* proj, int ld, int q_off, int k_off, int v_off, int g_off, int y_off, int inner, const float* w2,
+                     const float* b2, float inv_tau, float q_scale, const float* weight, float eps, float* out, int ldo, float* S,
+                     const int32_t* seqs, int n_seqs, int heads, int dim, int vdim, void* stream);
+int pgk_seq_gla_decays(const float* proj, int ld, int y_off, int inner, const float* w2, const float* b2, float inv_tau,
+                       const int32_t* seqs, int n_seqs, int max_rows, int heads, int dim, float* L, void* stream);
+int pgk_seq_gla_chunks(const float* proj, int ld, int q_off, int k_off, int v_off, int g_off, const float* L, float q_scale,
+                       const float* weight, float eps, float* out, int ldo, float* S, const int32_t* seqs, int n_seqs, int heads, int dim,
+                       int vdim, int chunk_begin, int chunks, float* workspace, void* stream);
+
 /* mixer_prep for layers whose q / k norm runs over the WHOLE projection: per token, q <- (q + q_bias) / rms(all heads x dim
  * of q) * (weight_offset + q_weight) in place (proj[t, 0 ..]), k the same from proj[t, k_off ..] with k_weight into the K
  * pages; the V pages receive k + k_bias as projected (before the norm).  Biases may be NULL; weights are [heads x dim] and
@@ -711,6 +734,12 @@ int pgk_seq_latent_prep(float* proj, int ld, int tokens, int q_rank, int kv_off,
                         const float* q_weight, const float* c_weight, float weight_offset, float eps, const double* inv_freq,
                         void* k_cache, int cache_dtype, const int32_t* table, int max_pages, int page_size,
                         const int32_t* slot, const int32_t* pos, void* stream);
+/* Query tails behind the absorbed queries and the cache row in one launch, with a factor on cosine and sine; rank 0: no cache row
+ * (the layer reads another one's).  Head h's tail: proj[t, h * q_head + q_tail] -> q_out[t, h * q_out_head + q_out_tail]. */
+int pgk_seq_latent_prep_heads(float* proj, int ld, int tokens, int q_head, int q_tail, int heads, float* q_out, int ldq_out,
+                              int q_out_head, int q_out_tail, int kv_off, int rank, int rot, int rot_dims, const float* c_weight,
+                              float weight_offset, float eps, const double* inv_freq, float rot_mult, void* k_cache, int cache_dtype,
+                              const int32_t* table, int max_pages, int page_size, const int32_t* slot, const int32_t* pos, void* stream);
 int pgk_seq_rope_heads(const float* src, int lds, int src_head, int src_off, float* dst, int ldd, int dst_head, int dst_off,
                        int tokens, int heads, int rot, int rot_dims, const double* inv_freq, const int32_t* pos, void* stream);
 /* v = x[src_rows ? src_rows[t] : t] + (add ? add[t] : 0); sum_out[t] = v when given (no gather then); r = v / sqrt(mean(v^2)
@@ -722,6 +751,15 @@ int pgk_rms_norm_rows_f32(const float* x, const int32_t* src_rows, const float* 
 int pgk_rms_norm_seam_f32(const float* y, const float* weight1, float offset1, float* x, const float* add, const float* weight2,
                           float offset2, float eps, float* h, int rows, int width, void* stream);
 /* x[t] = rms(table[tokens[t]]) * (weight_offset + weight), written to keep[t] as well when keep is not NULL */
+/* embedding rows times a constant */
+int pgk_embed_rows_scaled_f32(const void* table, int wdt, const int32_t* tokens, float scale, float* x, int n, int width, int vocab,
+                              void* stream);
+/* x[t] += base[t] + sum_k weights[t, k] parts[inv[t, k]] + sigmoid(gate_rows[t, gate_off]) shared[t] (each optional; no gate: factor
+ * 1), then h[t] = rms(x[t]) (weight_offset + weight) (h NULL: not wanted): a sublayer joins the residual stream and the next
+ * sublayer's norm is taken in one launch. */
+int pgk_rms_add_norm_f32(const float* base, const float* parts, const int32_t* inv, const float* weights, int top, const float* shared,
+                         const float* gate_rows, int ldg, int gate_off, float* x, const float* weight, float weight_offset, float eps,
+                         float* h, int rows, int width, void* stream);
 int pgk_embed_norm_rows_f32(const void* table, int wdt, const int32_t* tokens, const float* weight, float weight_offset, float eps,
                             float* x, float* keep, int n, int width, int vocab, void* stream);
 /* The general row GEMM: `batch` products over the same M rows, product b reading A columns from b * a_batch, matrix

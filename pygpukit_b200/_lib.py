@@ -162,6 +162,15 @@ _SIGS = {
                               i32, i32, i32, i32, i32, i32, i32, f32, f32, i32, vp, f32, i32, i32, vp, vp, vp, i32, i32, vp, vp, i32, vp],
     "pgk_rms_join_f32": [vp, vp, vp, vp, i32, vp, f32, vp, i32, i32, vp],
     "pgk_moe_route_logits": [vp, i32, i32, i32, i32, vp, i32, vp, vp, vp, vp, vp],
+    # gated linear attention (seq_gla.cu) and what its blocks share with others
+    "pgk_seq_gla_step": [vp, i32, i32, i32, i32, i32, i32, i32, vp, vp, f32, f32, vp, f32, vp, i32, vp, vp, i32, i32, i32, i32, vp],
+    "pgk_seq_gla_decays": [vp, i32, i32, i32, vp, vp, f32, vp, i32, i32, i32, i32, vp, vp],
+    "pgk_seq_gla_chunks": [vp, i32, i32, i32, i32, i32, vp, f32, vp, f32, vp, i32, vp, vp, i32, i32, i32, i32, i32, i32, vp, vp],
+    "pgk_seq_latent_prep_heads": [vp, i32, i32, i32, i32, i32, vp, i32, i32, i32, i32, i32, i32, i32, vp, f32, f32, vp, f32, vp, i32, vp,
+                                  i32, i32, vp, vp, vp],
+    "pgk_embed_rows_scaled_f32": [vp, i32, vp, f32, vp, i32, i32, i32, vp],
+    "pgk_rms_add_norm_f32": [vp, vp, vp, vp, i32, vp, vp, i32, i32, vp, vp, f32, f32, vp, i32, i32, vp],
+    "pgk_moe_route_sigmoid": [vp, i32, i32, i32, i32, vp, i32, i32, f32, i32, vp, vp, vp, vp, vp],
     # matrix memory with exponential gates (seq_mlstm.cu)
     "pgk_seq_mlstm_step": [vp, i32, i32, i32, i32, i32, i32, i32, vp, vp, f32, f32, vp, f32, vp, i32, vp, vp, vp, vp, i32, i32, i32, i32, vp],
     "pgk_seq_mlstm_gates": [vp, i32, i32, i32, vp, vp, f32, vp, vp, i32, i32, i32, vp, vp],
@@ -175,12 +184,14 @@ _RESTYPE = {"pgk_last_error": C.c_char_p, "pgk_launch_count": i64, "pgk_launch_c
             "pgk_sdpa_workspace_bytes": sz, "pgk_p2p_handle_bytes": sz, "pgk_p2p_ready": i32,
             "pgk_p2p_max_bytes": sz, "pgk_seq_heads_per_block": i32, "pgk_seq_queries_per_tile": i32,
             "pgk_seq_decode_heads_per_block": i32, "pgk_seq_linear_value_slice": i32, "pgk_seq_linear_chunk_tokens": i32,
-            "pgk_seq_mlstm_chunk_tokens": i32, "pgk_seq_mlstm_fused_finish": i32, "pgk_seq_mlstm_gate_floats": sz}
+            "pgk_seq_mlstm_chunk_tokens": i32, "pgk_seq_mlstm_fused_finish": i32, "pgk_seq_mlstm_gate_floats": sz,
+            "pgk_seq_gla_chunk_tokens": i32, "pgk_seq_gla_fused_finish": i32}
 _EXTRA = {"pgk_last_error": [], "pgk_launch_count": [], "pgk_launch_count_reset": [],
           "pgk_sdpa_workspace_bytes": [i32, i32, i32, i32], "pgk_p2p_handle_bytes": [], "pgk_p2p_ready": [], "pgk_p2p_max_bytes": [],
           "pgk_seq_heads_per_block": [i32, i32], "pgk_seq_queries_per_tile": [i32, i32],
           "pgk_seq_decode_heads_per_block": [], "pgk_seq_linear_value_slice": [i32, i32, i32, i32], "pgk_seq_linear_chunk_tokens": [],
-          "pgk_seq_mlstm_chunk_tokens": [], "pgk_seq_mlstm_fused_finish": [i32], "pgk_seq_mlstm_gate_floats": [i32, i32]}
+          "pgk_seq_mlstm_chunk_tokens": [], "pgk_seq_mlstm_fused_finish": [i32], "pgk_seq_mlstm_gate_floats": [i32, i32],
+          "pgk_seq_gla_chunk_tokens": [i32, i32], "pgk_seq_gla_fused_finish": [i32]}
 
 
 def load() -> C.CDLL:

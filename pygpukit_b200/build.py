@@ -54,6 +54,7 @@ SOURCES = {
     "seq_recurrent.cu": [],
     "seq_gated.cu": [],
     "seq_mlstm.cu": [],
+    "seq_gla.cu": [],
 }
 
 # groups of sources that link on their own (runtime.cu is in every library)
@@ -61,7 +62,7 @@ COMPONENTS = {
     "core": ["runtime.cu"],
     # token-major float32-activation models on the paged cache (llm/models/layered.py)
     "seq": ["runtime.cu", "seq_gemm.cu", "seq_attention.cu", "seq_layers.cu", "seq_latent.cu", "seq_recurrent.cu",
-            "seq_gated.cu", "seq_mlstm.cu"],
+            "seq_gated.cu", "seq_mlstm.cu", "seq_gla.cu"],
 }
 
 

@@ -8,6 +8,7 @@
 //                      scores themselves (renormalised on request); router outputs >= real_experts stand for experts without
 //                      matrices (`mat` = -1 for them)
 //   moe_route_logits   a bias on the logits, the `top` largest logits chosen, weights = softmax over the chosen ones only
+//   moe_route_sigmoid  scores sigmoid(logit), chosen by score + bias inside the best groups, weights = factor * score
 //   moe_combine_rows   out = sum_k w[t, k] * (parts row, or the token's own input row for an expert without matrices)
 //                      + sigmoid(gate logit) * shared expert row
 //   dyt_seam           a sublayer's result (plain rows, the two-branch join, or the expert sum) through the norm behind it into
@@ -193,6 +194,81 @@ __global__ void __launch_bounds__(ROUTE_WARPS * 32) moe_route_logits_kernel(Rout
     if (a.extra >= 0 && lane == 0) {
         a.idx[o + a.top] = a.extra;
         a.wt[o + a.top] = 1.f;
+        if (a.counts) a.rank[o + a.top] = atomicAdd(&a.counts[a.extra], 1);
+    }
+}
+
+// ---------------------------------------------------------------- router with sigmoid scores, a choice bias and group limits
+// One warp per token: s = sigmoid(z), choice = s + bias; groups of neighbours ranked by the sum of their two largest choices (a
+// group of one: its only one); the members of the gkeep best groups compete, the `top` largest choices win with weight scale * s.
+// With `extra` >= 0 every token also takes that matrix as its last slot, with weight sigmoid(z[E]) (z[E]: the gate of a shared
+// expert that rides in the experts' stack).
+struct RouteSigmoidArgs {
+    const float* z; int ldz, T, E, top, gcount, gkeep, extra;
+    const float* bias; float scale;
+    int* idx; float* wt; int* rank; int* counts;
+};
+
+__global__ void __launch_bounds__(ROUTE_WARPS * 32) moe_route_sigmoid_kernel(RouteSigmoidArgs a) {
+    extern __shared__ float sm[];
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    const int t = blockIdx.x * ROUTE_WARPS + warp;
+    if (t >= a.T) return;
+    float* s = sm + (size_t)warp * (2 * a.E + a.gcount);      // [E] scores
+    float* c = s + a.E;                                       // [E] choice scores; -inf once chosen or out of play
+    float* gs = c + a.E;                                      // [gcount]
+    const float* z = a.z + (size_t)t * a.ldz;
+    for (int e = lane; e < a.E; e += 32) {
+        const float p = sigmoid_f(z[e]);
+        s[e] = p;
+        c[e] = p + (a.bias ? a.bias[e] : 0.f);
+    }
+    __syncwarp();
+    if (a.gkeep < a.gcount) {
+        const int per = a.E / a.gcount;
+        for (int g = lane; g < a.gcount; g += 32) {
+            float b0 = -INFINITY, b1 = -INFINITY;
+            for (int j = 0; j < per; ++j) {
+                const float v = c[g * per + j];
+                b1 = fmaxf(b1, fminf(b0, v));
+                b0 = fmaxf(b0, v);
+            }
+            gs[g] = per > 1 ? b0 + b1 : b0;
+        }
+        __syncwarp();
+        for (int it = 0; it < a.gkeep; ++it) {                // kept groups are marked by +inf
+            float bv = -INFINITY; int bi = 0x7fffffff;
+            for (int g = lane; g < a.gcount; g += 32)
+                if (gs[g] != INFINITY && (gs[g] > bv || bi == 0x7fffffff)) { bv = gs[g]; bi = g; }
+            warp_argmax(bv, bi);
+            __syncwarp();
+            if (lane == 0) gs[bi] = INFINITY;
+            __syncwarp();
+        }
+        for (int e = lane; e < a.E; e += 32)
+            if (gs[e / per] != INFINITY) c[e] = -INFINITY;
+        __syncwarp();
+    }
+    const int slots = a.top + (a.extra >= 0 ? 1 : 0);
+    const size_t o = (size_t)t * slots;
+    for (int k = 0; k < a.top; ++k) {
+        float bv = -INFINITY; int bi = 0x7fffffff;
+        for (int e = lane; e < a.E; e += 32)
+            if (c[e] > bv) { bv = c[e]; bi = e; }
+        warp_argmax(bv, bi);
+        if (bi >= a.E) bi = 0;                                // logits that are not numbers: stay in range
+        __syncwarp();
+        if (lane == 0) {
+            c[bi] = -INFINITY;
+            a.idx[o + k] = bi;
+            a.wt[o + k] = a.scale * s[bi];
+            if (a.counts) a.rank[o + k] = atomicAdd(&a.counts[bi], 1);
+        }
+        __syncwarp();
+    }
+    if (a.extra >= 0 && lane == 0) {
+        a.idx[o + a.top] = a.extra;
+        a.wt[o + a.top] = sigmoid_f(z[a.E]);
         if (a.counts) a.rank[o + a.top] = atomicAdd(&a.counts[a.extra], 1);
     }
 }
@@ -631,6 +707,23 @@ int pgk_moe_route_logits(const float* logits, int ld, int tokens, int experts, i
     const size_t smem = (size_t)ROUTE_WARPS * experts * 4;
     PGK_REQUIRE(smem <= 48 * 1024, "moe_route_logits failed: too many experts (%d)", experts);
     PGK_CUDA(launch(moe_route_logits_kernel, dim3((tokens + ROUTE_WARPS - 1) / ROUTE_WARPS), dim3(ROUTE_WARPS * 32), smem,
+                    (cudaStream_t)stream, a));
+    return 0;
+}
+
+int pgk_moe_route_sigmoid(const float* logits, int ld, int tokens, int experts, int top, const float* bias, int group_count,
+                          int group_keep, float scale, int extra, int32_t* idx, float* weights, int32_t* rank, int32_t* counts,
+                          void* stream) {
+    PGK_REQUIRE(experts > 0 && top > 0 && top <= experts, "moe_route_sigmoid failed: top %d of %d experts", top, experts);
+    PGK_REQUIRE(group_count >= 1 && group_keep >= 1 && experts % group_count == 0 &&
+                (group_keep >= group_count || experts / group_count * group_keep >= top),
+                "moe_route_sigmoid failed: %d experts in %d groups, %d kept, top %d", experts, group_count, group_keep, top);
+    PGK_REQUIRE((rank == nullptr) == (counts == nullptr), "moe_route_sigmoid failed: ranks and counts come together");
+    if (tokens <= 0) return 0;
+    RouteSigmoidArgs a{logits, ld, tokens, experts, top, group_count, group_keep, extra, bias, scale, idx, weights, rank, counts};
+    const size_t smem = (size_t)ROUTE_WARPS * (2 * experts + group_count) * 4;
+    PGK_REQUIRE(smem <= 48 * 1024, "moe_route_sigmoid failed: too many experts (%d)", experts);
+    PGK_CUDA(launch(moe_route_sigmoid_kernel, dim3((tokens + ROUTE_WARPS - 1) / ROUTE_WARPS), dim3(ROUTE_WARPS * 32), smem,
                     (cudaStream_t)stream, a));
     return 0;
 }

@@ -12,7 +12,7 @@
 //     [M, N / 2]); scale then tanh cap (the logit head); clamped gate/up pairs g = min(gate, limit), u = clamp(up, +-limit),
 //     output g sigmoid(alpha g) (u + 1); C += column vector * product (layer scale and residual add in one pass);
 //     gelu_tanh(product) * gathered table entry (per-layer token inputs); squared ReLU; gate/up pairs with gelu_tanh(gate) * up;
-//     gelu_erf(product);
+//     gelu_erf(product); gelu_tanh(product); product * sigmoid(gate row's element);
 //   * batches: grid.z can also walk `batch` independent products whose A columns, matrices and C columns are a fixed number
 //     of elements apart (one product per attention head on slices of the same rows).
 #include "common.cuh"
@@ -33,7 +33,8 @@ struct GemmArgs {
     int lda, ldc, M, N, K;
     float scale, cap;
     const float* colv;        // epilogue 4: [N] factors of the accumulated product
-    const void* aux;          // epilogue 5: table [*, aux_ld] (float32 or bfloat16), entry (aux_rows[m], aux_off + n)
+    const void* aux;          // epilogue 5: table [*, aux_ld] (float32 or bfloat16), entry (aux_rows[m], aux_off + n);
+                              // epilogue 10: float32 gate rows, element (m, aux_off + C column)
     const int* aux_rows;
     int aux_ld, aux_off, aux_dt;
     long long a_z, c_z;       // batches: elements between the A columns / C columns of consecutive products
@@ -77,6 +78,12 @@ __device__ __forceinline__ void store_pair(const GemmArgs& a, int row, int col, 
         c0 *= c0; c1 *= c1;
     }
     if (EPI == 8) { c0 = gelu_erf_f(c0); c1 = gelu_erf_f(c1); }
+    if (EPI == 9) { c0 = gelu_tanh_f(c0); c1 = gelu_tanh_f(c1); }
+    if (EPI == 10) {         // the gate's columns are as far apart as the output's: `aux` moves with C from batch to batch
+        const float* g = (const float*)a.aux + (size_t)row * a.aux_ld + a.aux_off + col;
+        if (col < a.N) c0 *= 1.f / (1.f + expf(-g[0]));
+        if (col + 1 < a.N) c1 *= 1.f / (1.f + expf(-g[1]));
+    }
     float* p = a.C + (size_t)row * a.ldc + col;
     if (EPI == 4) {
         if (col < a.N) p[0] = fmaf(a.colv[col], c0, p[0]);
@@ -111,6 +118,7 @@ __global__ void __launch_bounds__(128) gemm_rows_bf16_kernel(GemmArgs a) {
     const int e = blockIdx.z;
     a.A += (size_t)e * a.a_z;
     a.C += (size_t)e * a.c_z;
+    if (EPI == 10) a.aux = (const float*)a.aux + (size_t)e * a.c_z;
     const int m_begin = a.group_off ? a.group_off[e] : 0;
     const int m_end = a.group_off ? a.group_off[e + 1] : a.M;
     const int m0 = m_begin + blockIdx.y * BM;
@@ -227,6 +235,7 @@ __global__ void __launch_bounds__(128) gemm_rows_f32_kernel(GemmArgs a) {
     const int e = blockIdx.z;
     a.A += (size_t)e * a.a_z;
     a.C += (size_t)e * a.c_z;
+    if (EPI == 10) a.aux = (const float*)a.aux + (size_t)e * a.c_z;
     const int m_begin = a.group_off ? a.group_off[e] : 0;
     const int m_end = a.group_off ? a.group_off[e + 1] : a.M;
     const int m0 = m_begin + blockIdx.y * BM;
@@ -314,6 +323,7 @@ __global__ void __launch_bounds__(FEW_MAX_WARPS * 32) gemm_few_rows_kernel(GemmA
     if (grp < 0) return;                                        // a row without a matrix (its output is formed elsewhere)
     a.A += (size_t)blockIdx.z * a.a_z;
     a.C += (size_t)blockIdx.z * a.c_z;
+    if (EPI == 10) a.aux = (const float*)a.aux + (size_t)blockIdx.z * a.c_z;
     const TW* W = (const TW*)a.W + (size_t)grp * a.w_stride;
     constexpr int VEC = WLoad<TW>::VEC;
     const bool vec = (a.K % VEC == 0) && (((uintptr_t)W & 15) == 0);
@@ -486,7 +496,7 @@ int pgk_gemm_rows_f32(const float* A, int lda, const int32_t* a_rows, const void
                       int epilogue, float scale, float cap, void* stream) {
     PGK_REQUIRE(wdt == 0 || wdt == 2, "gemm_rows_f32 failed: weights must be float32 (0) or bfloat16 (2), got %d", wdt);
     PGK_REQUIRE(N > 0 && K > 0 && M >= 0, "gemm_rows_f32 failed: invalid shape M=%d N=%d K=%d", M, N, K);
-    PGK_REQUIRE((epilogue >= 0 && epilogue <= 2) || epilogue == 7 || epilogue == 8, "gemm_rows_f32 failed: unknown epilogue %d", epilogue);
+    PGK_REQUIRE((epilogue >= 0 && epilogue <= 2) || (epilogue >= 6 && epilogue <= 9), "gemm_rows_f32 failed: unknown epilogue %d", epilogue);
     PGK_REQUIRE((epilogue != 1 && epilogue != 7) || N % 2 == 0, "gemm_rows_f32 failed: the gate/up epilogue needs an even N");
     const int G = group_off ? groups : 1;
     const int rows = group_off ? max_rows : M;
@@ -499,8 +509,10 @@ int pgk_gemm_rows_f32(const float* A, int lda, const int32_t* a_rows, const void
     }
     if (epilogue == 0) return launch_many<0>(a, wdt, G, rows, st);
     if (epilogue == 1) return launch_many<1>(a, wdt, G, rows, st);
+    if (epilogue == 6) return launch_many<6>(a, wdt, G, rows, st);
     if (epilogue == 7) return launch_many<7>(a, wdt, G, rows, st);
     if (epilogue == 8) return launch_many<8>(a, wdt, G, rows, st);
+    if (epilogue == 9) return launch_many<9>(a, wdt, G, rows, st);
     return launch_many<2>(a, wdt, G, rows, st);
 }
 
@@ -513,15 +525,17 @@ int pgk_gemm_few_rows_f32(const float* A, int lda, const int32_t* a_rows, const 
     PGK_REQUIRE(N > 0 && K > 0 && M >= 0, "gemm_few_rows_f32 failed: invalid shape M=%d N=%d K=%d", M, N, K);
     PGK_REQUIRE(rows_per_block >= 1 && rows_per_block <= RMAX, "gemm_few_rows_f32 failed: 1..%d rows per block", RMAX);
     PGK_REQUIRE((size_t)rows_per_block * K * 4 <= 200 * 1024, "gemm_few_rows_f32 failed: %d rows of K=%d do not fit shared memory", rows_per_block, K);
-    PGK_REQUIRE((epilogue >= 0 && epilogue <= 2) || epilogue == 7 || epilogue == 8, "gemm_few_rows_f32 failed: unknown epilogue %d", epilogue);
+    PGK_REQUIRE((epilogue >= 0 && epilogue <= 2) || (epilogue >= 6 && epilogue <= 9), "gemm_few_rows_f32 failed: unknown epilogue %d", epilogue);
     PGK_REQUIRE((epilogue != 1 && epilogue != 7) || N % 2 == 0, "gemm_few_rows_f32 failed: the gate/up epilogue needs an even N");
     if (M == 0) return 0;
     GemmArgs a{A, a_rows, W, C, nullptr, row_group, w_group_stride, lda, ldc, M, N, K, scale, cap, nullptr, nullptr, nullptr, 0, 0, 0, 0, 0};
     cudaStream_t st = (cudaStream_t)stream;
     if (epilogue == 0) return launch_few<0>(a, wdt, rows_per_block, st);
     if (epilogue == 1) return launch_few<1>(a, wdt, rows_per_block, st);
+    if (epilogue == 6) return launch_few<6>(a, wdt, rows_per_block, st);
     if (epilogue == 7) return launch_few<7>(a, wdt, rows_per_block, st);
     if (epilogue == 8) return launch_few<8>(a, wdt, rows_per_block, st);
+    if (epilogue == 9) return launch_few<9>(a, wdt, rows_per_block, st);
     return launch_few<2>(a, wdt, rows_per_block, st);
 }
 
@@ -535,10 +549,11 @@ int pgk_gemm_seq_f32(const float* A, int lda, long long a_batch, const void* W, 
                      void* stream) {
     PGK_REQUIRE(wdt == 0 || wdt == 2, "gemm_seq_f32 failed: weights must be float32 (0) or bfloat16 (2), got %d", wdt);
     PGK_REQUIRE(N > 0 && K > 0 && M >= 0 && batch >= 1, "gemm_seq_f32 failed: invalid shape M=%d N=%d K=%d batch=%d", M, N, K, batch);
-    PGK_REQUIRE(epilogue >= 0 && epilogue <= 8, "gemm_seq_f32 failed: unknown epilogue %d", epilogue);
+    PGK_REQUIRE(epilogue >= 0 && epilogue <= 10, "gemm_seq_f32 failed: unknown epilogue %d", epilogue);
     PGK_REQUIRE((epilogue != 1 && epilogue != 3 && epilogue != 7) || N % 2 == 0, "gemm_seq_f32 failed: a gate/up epilogue needs an even N");
     PGK_REQUIRE(epilogue != 4 || col_scale, "gemm_seq_f32 failed: the scaled-accumulate epilogue needs its column factors");
     PGK_REQUIRE(epilogue != 5 || (aux && aux_rows && (aux_dtype == 0 || aux_dtype == 2)), "gemm_seq_f32 failed: the gather epilogue needs its table and rows");
+    PGK_REQUIRE(epilogue != 10 || (aux && aux_dtype == 0), "gemm_seq_f32 failed: the gate epilogue needs its float32 rows");
     PGK_REQUIRE(rows_per_block >= 0 && rows_per_block <= RMAX, "gemm_seq_f32 failed: 0..%d rows per block", RMAX);
     PGK_REQUIRE(rows_per_block == 0 || (size_t)rows_per_block * K * 4 <= 200 * 1024, "gemm_seq_f32 failed: %d rows of K=%d do not fit shared memory", rows_per_block, K);
     if (M == 0) return 0;
@@ -554,7 +569,9 @@ int pgk_gemm_seq_f32(const float* A, int lda, long long a_batch, const void* W, 
             case 5: return launch_few<5>(a, wdt, rows_per_block, st, batch);
             case 6: return launch_few<6>(a, wdt, rows_per_block, st, batch);
             case 7: return launch_few<7>(a, wdt, rows_per_block, st, batch);
-            default: return launch_few<8>(a, wdt, rows_per_block, st, batch);
+            case 8: return launch_few<8>(a, wdt, rows_per_block, st, batch);
+            case 9: return launch_few<9>(a, wdt, rows_per_block, st, batch);
+            default: return launch_few<10>(a, wdt, rows_per_block, st, batch);
         }
     }
     switch (epilogue) {
@@ -566,7 +583,9 @@ int pgk_gemm_seq_f32(const float* A, int lda, long long a_batch, const void* W, 
         case 5: return launch_many<5>(a, wdt, batch, M, st);
         case 6: return launch_many<6>(a, wdt, batch, M, st);
         case 7: return launch_many<7>(a, wdt, batch, M, st);
-        default: return launch_many<8>(a, wdt, batch, M, st);
+        case 8: return launch_many<8>(a, wdt, batch, M, st);
+        case 9: return launch_many<9>(a, wdt, batch, M, st);
+        default: return launch_many<10>(a, wdt, batch, M, st);
     }
 }
 

@@ -8,6 +8,8 @@
 //
 //   latent_prep:  per token, on the fused projection row [dq (q_rank) | dkv (rank + rot) | ...]: RMS norm of dq in place,
 //                 RMS norm of the latent into the cache row, rotation of the shared key part into the cache row.
+//                 The cache row and the query tails (below) can be written by one launch (latent_prep_heads), which also covers
+//                 layers without a latent of their own (no cache row) and a factor on cosine and sine.
 //   rope_heads:   rotates the `rot` tail of every query head and places it behind the head's absorbed query.
 //
 // Rotation: dimension 2i is paired with 2i + 1 (interleaved), angle = position * inv_freq[i]; the angle is formed and
@@ -50,12 +52,11 @@ struct LatentPrepArgs {
     const double* inv_freq;
     void* kc; const int* table; int max_pages, PS;
     const int* slot; const int* pos;
+    float mult;                                       // factor on cosine and sine
 };
 
 template <typename TC>
-__global__ void __launch_bounds__(256) latent_prep_kernel(LatentPrepArgs a) {
-    __shared__ float red[8];
-    const int t = blockIdx.x;
+__device__ __forceinline__ void latent_row(const LatentPrepArgs& a, int t, float* red) {
     float* dq = a.proj + (size_t)t * a.ld;
     const float* dkv = dq + a.kv_off;
     float sq = 0.f, sc = 0.f;
@@ -74,6 +75,7 @@ __global__ void __launch_bounds__(256) latent_prep_kernel(LatentPrepArgs a) {
     for (int i = threadIdx.x; i < a.rot_dims / 2; i += blockDim.x) {
         float sn, cs;
         angle_sincos(pos, a.inv_freq[i], sn, cs);
+        sn *= a.mult; cs *= a.mult;
         const float u = kr[2 * i], v = kr[2 * i + 1];
         cstore<TC>(dst + a.rank + 2 * i, u * cs - v * sn);
         cstore<TC>(dst + a.rank + 2 * i + 1, v * cs + u * sn);
@@ -81,20 +83,29 @@ __global__ void __launch_bounds__(256) latent_prep_kernel(LatentPrepArgs a) {
     for (int i = a.rot_dims + threadIdx.x; i < a.rot; i += blockDim.x) cstore<TC>(dst + a.rank + i, kr[i]);
 }
 
+template <typename TC>
+__global__ void __launch_bounds__(256) latent_prep_kernel(LatentPrepArgs a) {
+    __shared__ float red[8];
+    latent_row<TC>(a, blockIdx.x, red);
+}
+
 struct RopeHeadsArgs {
     const float* src; int lds, src_head, src_off;     // head h's tail starts at src[t, h * src_head + src_off]
     float* dst; int ldd, dst_head, dst_off;
     int H, rot, rot_dims;
     const double* inv_freq; const int* pos;
+    float mult;
 };
 
-__global__ void __launch_bounds__(256) rope_heads_kernel(RopeHeadsArgs a) {
-    const int t = blockIdx.x, pos = a.pos[t];
+// the tails of token t, dealt to `parts` blocks
+__device__ __forceinline__ void rope_tails(const RopeHeadsArgs& a, int t, int part, int parts) {
+    const int pos = a.pos[t], first = part * blockDim.x + threadIdx.x, stride = parts * blockDim.x;
     const int half = a.rot_dims / 2;
-    for (int i = threadIdx.x; i < a.H * half; i += blockDim.x) {
+    for (int i = first; i < a.H * half; i += stride) {
         const int h = i / half, p = i - h * half;
         float sn, cs;
         angle_sincos(pos, a.inv_freq[p], sn, cs);
+        sn *= a.mult; cs *= a.mult;
         const float* s = a.src + (size_t)t * a.lds + (size_t)h * a.src_head + a.src_off;
         float* d = a.dst + (size_t)t * a.ldd + (size_t)h * a.dst_head + a.dst_off;
         const float u = s[2 * p], v = s[2 * p + 1];
@@ -102,10 +113,20 @@ __global__ void __launch_bounds__(256) rope_heads_kernel(RopeHeadsArgs a) {
         d[2 * p + 1] = v * cs + u * sn;
     }
     const int rest = a.rot - a.rot_dims;
-    for (int i = threadIdx.x; i < a.H * rest; i += blockDim.x) {
+    for (int i = first; i < a.H * rest; i += stride) {
         const int h = i / rest, p = a.rot_dims + (i - h * rest);
         a.dst[(size_t)t * a.ldd + (size_t)h * a.dst_head + a.dst_off + p] = a.src[(size_t)t * a.lds + (size_t)h * a.src_head + a.src_off + p];
     }
+}
+
+__global__ void __launch_bounds__(256) rope_heads_kernel(RopeHeadsArgs a) { rope_tails(a, blockIdx.x, 0, 1); }
+
+// blocks (t, 0 .. parts - 1): query tails; block (t, parts), when there is one: the cache row
+template <typename TC>
+__global__ void __launch_bounds__(256) latent_prep_heads_kernel(LatentPrepArgs p, RopeHeadsArgs a, int parts) {
+    __shared__ float red[8];
+    if ((int)blockIdx.y < parts) rope_tails(a, blockIdx.x, blockIdx.y, parts);
+    else latent_row<TC>(p, blockIdx.x, red);
 }
 
 }  // namespace
@@ -121,7 +142,7 @@ int pgk_seq_latent_prep(float* proj, int ld, int tokens, int q_rank, int kv_off,
                 "seq_latent_prep failed: rank %d, rotated part %d of which %d turn", rank, rot, rot_dims);
     if (tokens <= 0) return 0;
     LatentPrepArgs a{proj, ld, q_rank, rank, rot, rot_dims, kv_off, q_weight, c_weight, weight_offset, eps, inv_freq, k_cache,
-                     table, max_pages, page_size, slot, pos};
+                     table, max_pages, page_size, slot, pos, 1.f};
     if (cache_dtype == 2) PGK_CUDA(launch(latent_prep_kernel<uint16_t>, dim3(tokens), dim3(256), 0, (cudaStream_t)stream, a));
     else PGK_CUDA(launch(latent_prep_kernel<float>, dim3(tokens), dim3(256), 0, (cudaStream_t)stream, a));
     return 0;
@@ -132,8 +153,29 @@ int pgk_seq_rope_heads(const float* src, int lds, int src_head, int src_off, flo
     PGK_REQUIRE(heads > 0 && rot >= 0 && rot_dims >= 0 && rot_dims <= rot && rot_dims % 2 == 0,
                 "seq_rope_heads failed: %d heads, rotated part %d of which %d turn", heads, rot, rot_dims);
     if (tokens <= 0 || rot == 0) return 0;
-    RopeHeadsArgs a{src, lds, src_head, src_off, dst, ldd, dst_head, dst_off, heads, rot, rot_dims, inv_freq, pos};
+    RopeHeadsArgs a{src, lds, src_head, src_off, dst, ldd, dst_head, dst_off, heads, rot, rot_dims, inv_freq, pos, 1.f};
     PGK_CUDA(launch(rope_heads_kernel, dim3(tokens), dim3(256), 0, (cudaStream_t)stream, a));
+    return 0;
+}
+
+/* rank 0: no cache row (a layer that reads another one's) */
+int pgk_seq_latent_prep_heads(float* proj, int ld, int tokens, int q_head, int q_tail, int heads, float* q_out, int ldq_out,
+                              int q_out_head, int q_out_tail, int kv_off, int rank, int rot, int rot_dims, const float* c_weight,
+                              float weight_offset, float eps, const double* inv_freq, float rot_mult, void* k_cache, int cache_dtype,
+                              const int32_t* table, int max_pages, int page_size, const int32_t* slot, const int32_t* pos, void* stream) {
+    PGK_REQUIRE(cache_dtype == 0 || cache_dtype == 2, "seq_latent_prep_heads failed: the cache is float32 (0) or bfloat16 (2), got %d", cache_dtype);
+    PGK_REQUIRE(heads > 0 && rank >= 0 && rot >= 0 && rot_dims >= 0 && rot_dims <= rot && rot_dims % 2 == 0,
+                "seq_latent_prep_heads failed: rank %d, rotated part %d of which %d turn", rank, rot, rot_dims);
+    PGK_REQUIRE(rank == 0 || (k_cache && c_weight), "seq_latent_prep_heads failed: the cache row needs its array and its norm weight");
+    if (tokens <= 0) return 0;
+    LatentPrepArgs p{proj, ld, 0, rank, rot, rot_dims, kv_off, nullptr, c_weight, weight_offset, eps, inv_freq, k_cache,
+                     table, max_pages, page_size, slot, pos, rot_mult};
+    RopeHeadsArgs a{proj, ld, q_head, q_tail, q_out, ldq_out, q_out_head, q_out_tail, heads, rot, rot_dims, inv_freq, pos, rot_mult};
+    const int parts = rot == 0 ? 0 : (tokens <= 32 ? (heads * rot / 2 + 255) / 256 : 1);
+    const dim3 grid(tokens, parts + (rank > 0 ? 1 : 0));
+    if (grid.y == 0) return 0;
+    if (cache_dtype == 2) PGK_CUDA(launch(latent_prep_heads_kernel<uint16_t>, grid, dim3(256), 0, (cudaStream_t)stream, p, a, parts));
+    else PGK_CUDA(launch(latent_prep_heads_kernel<float>, grid, dim3(256), 0, (cudaStream_t)stream, p, a, parts));
     return 0;
 }
 

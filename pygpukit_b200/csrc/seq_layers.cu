@@ -15,7 +15,7 @@ template <> __device__ __forceinline__ float wload<float>(const float* p) { retu
 template <> __device__ __forceinline__ float wload<uint16_t>(const uint16_t* p) { return bf16_bits_to_f32(*p); }
 
 template <typename TW>
-__global__ void __launch_bounds__(256) embed_rows_kernel(const TW* table, const int* tok, float* x, int W, int vocab) {
+__global__ void __launch_bounds__(256) embed_rows_kernel(const TW* table, const int* tok, float* x, int W, int vocab, float scale) {
     const int t = blockIdx.x;
     int id = tok[t];
     id = id < 0 ? 0 : (id >= vocab ? vocab - 1 : id);
@@ -26,7 +26,7 @@ __global__ void __launch_bounds__(256) embed_rows_kernel(const TW* table, const 
     for (int j = 0; j < 4; ++j) v[j] = i0 + j < W ? wload<TW>(src + i0 + j) : 0.f;
 #pragma unroll
     for (int j = 0; j < 4; ++j)
-        if (i0 + j < W) x[(size_t)t * W + i0 + j] = v[j];
+        if (i0 + j < W) x[(size_t)t * W + i0 + j] = v[j] * scale;
 }
 
 __device__ __forceinline__ float block_sum256(float v, float* red) {
@@ -237,6 +237,104 @@ __global__ void __launch_bounds__(1024) rms_join_kernel(RmsJoinArgs a) {
     }
 }
 
+// The seam in front of a pre-norm sublayer: x[t] += base[t] (may be absent) + sum_k w[t, k] * parts[inv[t, k]] + sigmoid(gate[t]) *
+// shared[t] (the sublayer before it joins the residual stream), written back, then h[t] = rms(x[t]) * (off + weight) (h NULL: not
+// wanted).  With nothing to add it is the norm alone.  Threads and registers as in rms_join.
+struct RmsAddNormArgs {
+    const float* base; const float* parts; const int* inv; const float* w; int top;
+    const float* shared; const float* gate; int ldg, gate_off;
+    float* x; const float* weight; float off, eps;
+    float* h; int W;
+};
+
+template <bool VEC>
+__global__ void __launch_bounds__(1024) rms_add_norm_kernel(RmsAddNormArgs a) {
+    __shared__ float red[32];
+    __shared__ float wk[TOPMAX];
+    __shared__ long long pk[TOPMAX];
+    constexpr int E = VEC ? 4 : 1;
+    const int t = blockIdx.x, tid = threadIdx.x, nt = blockDim.x, top = a.top;
+    const size_t o = (size_t)t * a.W;
+    const bool adds = a.base || top > 0 || a.shared;
+    const float sg = a.shared ? (a.gate ? 1.f / (1.f + expf(-a.gate[(size_t)t * a.ldg + a.gate_off])) : 1.f) : 0.f;
+    float v[JOIN_MAX], wv[JOIN_MAX];
+#pragma unroll
+    for (int j = 0; j < JOIN_MAX / E; ++j) {          // what depends on nothing but the row goes out first
+        const int i = (tid + j * nt) * E;
+        if (i >= a.W) continue;
+        if (VEC) {
+            *(float4*)&v[j * E] = *(const float4*)(a.x + o + i);
+            if (a.h) *(float4*)&wv[j * E] = *(const float4*)(a.weight + i);
+            if (a.base) {
+                const float4 b = *(const float4*)(a.base + o + i);
+                v[j * E] += b.x; v[j * E + E / 4] += b.y; v[j * E + E / 2] += b.z; v[j * E + E - 1] += b.w;
+            }
+            if (a.shared) {
+                const float4 s = *(const float4*)(a.shared + o + i);
+                v[j * E] = fmaf(sg, s.x, v[j * E]); v[j * E + E / 4] = fmaf(sg, s.y, v[j * E + E / 4]);
+                v[j * E + E / 2] = fmaf(sg, s.z, v[j * E + E / 2]); v[j * E + E - 1] = fmaf(sg, s.w, v[j * E + E - 1]);
+            }
+        } else {
+            v[j] = a.x[o + i] + (a.base ? a.base[o + i] : 0.f);
+            if (a.shared) v[j] = fmaf(sg, a.shared[o + i], v[j]);
+            if (a.h) wv[j] = a.weight[i];
+        }
+    }
+    for (int k0 = 0; k0 < top; k0 += TOPMAX) {
+        const int kn = min(TOPMAX, top - k0);
+        __syncthreads();
+        if (tid < kn) {
+            wk[tid] = a.w[(size_t)t * top + k0 + tid];
+            pk[tid] = (long long)a.inv[(size_t)t * top + k0 + tid] * a.W;
+        }
+        __syncthreads();
+#pragma unroll
+        for (int j = 0; j < JOIN_MAX / E; ++j) {
+            const int i = (tid + j * nt) * E;
+            if (i >= a.W) continue;
+#pragma unroll 4
+            for (int k = 0; k < kn; ++k) {
+                if (VEC) {
+                    const float4 p = *(const float4*)(a.parts + pk[k] + i);
+                    const float pp[4] = {p.x, p.y, p.z, p.w};
+#pragma unroll
+                    for (int e = 0; e < E; ++e) v[j * E + e] = fmaf(wk[k], pp[e], v[j * E + e]);
+                } else {
+                    v[j] = fmaf(wk[k], a.parts[pk[k] + i], v[j]);
+                }
+            }
+        }
+    }
+    float q = 0.f;
+#pragma unroll
+    for (int j = 0; j < JOIN_MAX / E; ++j) {
+        const int i = (tid + j * nt) * E;
+        if (i >= a.W) continue;
+#pragma unroll
+        for (int e = 0; e < E; ++e) q = fmaf(v[j * E + e], v[j * E + e], q);
+        if (adds) {
+            if (VEC) *(float4*)(a.x + o + i) = *(const float4*)&v[j * E];
+            else a.x[o + i] = v[j];
+        }
+    }
+    if (!a.h) return;
+    q = warp_sum(q);
+    if ((tid & 31) == 0) red[tid >> 5] = q;
+    __syncthreads();
+    float s = 0.f;
+    for (int i = 0; i < (nt >> 5); ++i) s += red[i];
+    const float inv = 1.f / sqrtf(s / (float)a.W + a.eps);
+#pragma unroll
+    for (int j = 0; j < JOIN_MAX / E; ++j) {
+        const int i = (tid + j * nt) * E;
+        if (i >= a.W) continue;
+#pragma unroll
+        for (int e = 0; e < E; ++e) v[j * E + e] = v[j * E + e] * inv * (a.off + wv[j * E + e]);
+        if (VEC) *(float4*)(a.h + o + i) = *(const float4*)&v[j * E];
+        else a.h[o + i] = v[j];
+    }
+}
+
 // x[t] = rms(table[tokens[t]]) * (off + w), copied to keep[t] as well when given: embedding, its norm and the kept copy
 template <typename TW>
 __global__ void __launch_bounds__(256) embed_norm_rows_kernel(const TW* table, const int* tok, const float* w, float off, float eps,
@@ -365,10 +463,15 @@ __global__ void __launch_bounds__(1024) moe_lists_kernel(int* counts, int* offse
 extern "C" {
 
 int pgk_embed_rows_f32(const void* table, int wdt, const int32_t* tokens, float* x, int n, int width, int vocab, void* stream) {
+    return pgk_embed_rows_scaled_f32(table, wdt, tokens, 1.f, x, n, width, vocab, stream);
+}
+
+int pgk_embed_rows_scaled_f32(const void* table, int wdt, const int32_t* tokens, float scale, float* x, int n, int width, int vocab,
+                              void* stream) {
     PGK_REQUIRE(wdt == 0 || wdt == 2, "embed_rows_f32 failed: table must be float32 (0) or bfloat16 (2), got %d", wdt);
     if (n <= 0) return 0;
-    if (wdt == 2) PGK_CUDA(launch(embed_rows_kernel<uint16_t>, dim3(n, (width + 1023) / 1024), dim3(256), 0, (cudaStream_t)stream, (const uint16_t*)table, tokens, x, width, vocab));
-    else PGK_CUDA(launch(embed_rows_kernel<float>, dim3(n, (width + 1023) / 1024), dim3(256), 0, (cudaStream_t)stream, (const float*)table, tokens, x, width, vocab));
+    if (wdt == 2) PGK_CUDA(launch(embed_rows_kernel<uint16_t>, dim3(n, (width + 1023) / 1024), dim3(256), 0, (cudaStream_t)stream, (const uint16_t*)table, tokens, x, width, vocab, scale));
+    else PGK_CUDA(launch(embed_rows_kernel<float>, dim3(n, (width + 1023) / 1024), dim3(256), 0, (cudaStream_t)stream, (const float*)table, tokens, x, width, vocab, scale));
     return 0;
 }
 
@@ -434,6 +537,24 @@ int pgk_rms_join_f32(const float* base, const float* parts, const int32_t* inv, 
     while ((long long)nt * JOIN_MAX < width && nt < 1024) nt += 32;
     if (vec) PGK_CUDA(launch(rms_join_kernel<true>, dim3(rows), dim3(nt), 0, (cudaStream_t)stream, a));
     else PGK_CUDA(launch(rms_join_kernel<false>, dim3(rows), dim3(nt), 0, (cudaStream_t)stream, a));
+    return 0;
+}
+
+int pgk_rms_add_norm_f32(const float* base, const float* parts, const int32_t* inv, const float* weights, int top, const float* shared,
+                         const float* gate_rows, int ldg, int gate_off, float* x, const float* weight, float weight_offset, float eps,
+                         float* h, int rows, int width, void* stream) {
+    PGK_REQUIRE(width > 0 && width <= 1024 * JOIN_MAX, "rms_add_norm_f32 failed: width %d out of range", width);
+    PGK_REQUIRE(x && top >= 0 && (top == 0 || (parts && inv && weights)) && (!h || weight), "rms_add_norm_f32 failed: a missing operand");
+    if (rows <= 0 || (!h && !base && top == 0 && !shared)) return 0;
+    RmsAddNormArgs a{base, parts, inv, weights, top, shared, gate_rows, ldg, gate_off, x, weight, weight_offset, eps, h, width};
+    const bool vec = width % 4 == 0 && (((uintptr_t)base | (uintptr_t)parts | (uintptr_t)shared | (uintptr_t)x | (uintptr_t)weight | (uintptr_t)h) & 15) == 0;
+    const int units = vec ? width / 4 : width;
+    int nt = rows <= 32 ? (units + 31) / 32 * 32 : (units + 63) / 64 * 32;      // few rows: one group per thread
+    if (nt < 64) nt = 64;
+    if (nt > 1024) nt = 1024;
+    while ((long long)nt * JOIN_MAX < width && nt < 1024) nt += 32;
+    if (vec) PGK_CUDA(launch(rms_add_norm_kernel<true>, dim3(rows), dim3(nt), 0, (cudaStream_t)stream, a));
+    else PGK_CUDA(launch(rms_add_norm_kernel<false>, dim3(rows), dim3(nt), 0, (cudaStream_t)stream, a));
     return 0;
 }
 

@@ -7,6 +7,8 @@ tensor-name patterns belong to checkpoint loading, which is out of scope: SURVEY
 """
 from __future__ import annotations
 
+import math
+
 from dataclasses import dataclass
 from typing import Literal
 
@@ -329,6 +331,34 @@ class RotarySpec:
 
 
 @dataclass(frozen=True)
+class YarnSpec:
+    """Position scaling by frequency (YaRN): pairs that turn more than `fast` times within `original` positions keep their
+    frequency, pairs that turn fewer than `slow` times have it divided by `factor`, and between the two it is mixed along a ramp
+    over the pair index; cosine and sine are multiplied by 0.1 ln(factor) + 1."""
+    factor: float
+    original: float
+    fast: float
+    slow: float
+
+    def _index(self, turns: float, dims: int, base: float) -> float:
+        """the (fractional) pair index whose angle makes `turns` turns within `original` positions"""
+        return dims * math.log(self.original / (2.0 * math.pi * turns)) / (2.0 * math.log(base))
+
+    def inv_freq(self, dims: int, base: float) -> list[float]:
+        lo = max(math.floor(self._index(self.fast, dims, base)), 0)
+        hi = min(math.ceil(self._index(self.slow, dims, base)), dims - 1)
+        out = []
+        for i in range(dims // 2):
+            f, ramp = base ** (-2.0 * i / dims), min(max((i - lo) / max(hi - lo, 0.001), 0.0), 1.0)
+            out.append(f / self.factor * ramp + f * (1.0 - ramp))
+        return out
+
+    @property
+    def mult(self) -> float:
+        return 0.1 * math.log(self.factor) + 1.0
+
+
+@dataclass(frozen=True)
 class LinearMixerSpec:
     """Linear attention with a fixed decay per head and a float32 state per sequence instead of cache pages:
     S_t = decay_h S_(t-1) + k_t v_t^T, o_t = S_t^T q_t; H heads, keys of size `dim`, values of size `vdim`.
@@ -482,6 +512,42 @@ class MatrixLSTMSpec:
 
 
 @dataclass(frozen=True)
+class GLAMixerSpec:
+    """Gated linear attention with a float32 state per sequence: per head S_t = diag(a_t) S_(t-1) + k_t v_t^T, o_t = S_t^T q_t with
+    q times dim^-1/2 and a decay per head and key channel, a = sigmoid(W_2 (W_1 h) + b)^(1 / tau), through an inner size
+    `gate_rank` (0: not known yet; the loader takes it from the stored matrices).  Every head's output is divided by its root mean
+    square, multiplied by a weight vector shared by the heads and by silu of a gate projection."""
+    heads: int
+    dim: int
+    vdim: int
+    tau: float
+    gate_rank: int = 0
+
+    kind = "gla"
+    kv_heads = 0
+    chunk = 0
+    window = 0
+    keep_first = 0
+    pool = 0
+
+    @property
+    def proj_cols(self) -> int:
+        """columns of the fused projection [q | k | v | gate | inner decay columns]"""
+        return 2 * self.heads * self.dim + 2 * self.heads * self.vdim + self.gate_rank
+
+    @property
+    def attn_cols(self) -> int:
+        return self.heads * self.vdim
+
+    def cache_shape(self) -> tuple[int, int, int]:
+        return (0, 0, 0)                 # no cache pages
+
+    @property
+    def state_shapes(self) -> tuple:
+        return (self.heads * self.dim * self.vdim,)
+
+
+@dataclass(frozen=True)
 class ParallelMixerSpec:
     """Two mixers side by side on the same input (an attention mixer with cache pages and a mixer with a state).  `join`
     "sum": left_scale * left + right_scale * right, one output projection over both sides' heads; "rms_mean": each side has
@@ -537,8 +603,10 @@ class LatentMixerSpec:
     """Latent attention: queries through a latent of size `q_rank` (0: projected directly), keys and values through one
     latent of size `kv_rank` per position plus `rot_dim` rotated key dimensions shared by the heads.  Per head `dim`
     unrotated + `rot_dim` rotated query/key dimensions and `vdim` value dimensions; the rotation turns the first
-    `rot_dims` of the rotated part (interleaved pairs, base `rot_base`); causal; `sink` and the per-head gate as in
-    AttentionMixerSpec.  Only the latent and the rotated key part are cached."""
+    `rot_dims` of the rotated part (interleaved pairs, base `rot_base`, frequencies scaled by `yarn`); causal; `window`, `sink` and
+    the per-head gate as in AttentionMixerSpec (a gate of one number per element multiplies the heads' values, behind W_uv).
+    Only the latent and the rotated key part are cached.  `kv_from` >= 0: the layer has no latent of its own and reads the one
+    that layer `kv_from` has cached, with its own up-projections, queries and window."""
     heads: int
     dim: int
     rot_dim: int
@@ -551,13 +619,24 @@ class LatentMixerSpec:
     sink: str = "learned"
     out_gate: bool = True
     gate_per_head: bool = True
+    window: int = 0
+    yarn: "YarnSpec | None" = None
+    kv_from: int = -1
 
     kind = "latent_attention"
     kv_heads = 1
     chunk = 0
-    window = 0
     keep_first = 0
     state_shapes = ()
+
+    @property
+    def q_cols(self) -> int:
+        """columns of the fused projection that belong to the query: its latent, or the heads themselves"""
+        return self.q_rank if self.q_rank > 0 else self.heads * (self.dim + self.rot_dim)
+
+    @property
+    def kv_cols(self) -> int:
+        return self.kv_rank + self.rot_dim if self.kv_from < 0 else 0
 
     @property
     def gate_cols(self) -> int:
@@ -565,8 +644,8 @@ class LatentMixerSpec:
 
     @property
     def proj_cols(self) -> int:
-        """columns of the fused projection [query latent | key/value latent + rotated key | gate]"""
-        return self.q_rank + self.kv_rank + self.rot_dim + self.gate_cols
+        """columns of the fused projection [query (latent) | key/value latent + rotated key | gate]"""
+        return self.q_cols + self.kv_cols + self.gate_cols
 
     @property
     def attn_cols(self) -> int:
@@ -574,10 +653,19 @@ class LatentMixerSpec:
         return self.heads * (self.kv_rank + self.rot_dim)
 
     def cache_shape(self) -> tuple[int, int, int]:
+        if self.kv_from >= 0:
+            return (0, 0, 0)                                 # another layer's pages
         return (1, self.kv_rank + self.rot_dim, 0)          # value rows are a prefix of the key rows
 
+    @property
+    def rot_mult(self) -> float:
+        """factor on cosine and sine"""
+        return self.yarn.mult if self.yarn is not None else 1.0
+
     def inv_freq(self) -> list[float]:
-        """angle per position of pair i = rot_base^(-2 i / rot_dims)"""
+        """angle per position of pair i = rot_base^(-2 i / rot_dims), scaled by `yarn`"""
+        if self.yarn is not None:
+            return self.yarn.inv_freq(self.rot_dims, self.rot_base)
         return [self.rot_base ** (-2.0 * i / self.rot_dims) for i in range(self.rot_dims // 2)]
 
 
@@ -586,7 +674,7 @@ class DenseSpec:
     """Gated dense feed-forward: g = W_gate h, u = W_up h, output W_down act(g, u).  activation "silu": silu(g) u;
     "gelu_tanh": gelu(g) u with the tanh form;
     "clamped_swish": g <- min(g, limit), u <- clamp(u, -limit, limit), g sigmoid(alpha g) (u + 1).  "relu2" has no gate:
-    W_down max(W_up h, 0)^2.  "polynorm" has no gate either: W_down (a N(z) + b N(z^2) + c N(z^3) + e) with z = W_up h,
+    W_down max(W_up h, 0)^2; "gelu_tanh_up" neither: W_down gelu(W_up h), the tanh form.  "polynorm" has no gate either: W_down (a N(z) + b N(z^2) + c N(z^3) + e) with z = W_up h,
     powers element by element, N = division by the root mean square over the ff values, and four learned numbers."""
     ff: int
     activation: str = "silu"
@@ -607,8 +695,10 @@ class MoESpec:
     the weights are the scores themselves (`renorm` False) -- the last `identity` outputs stand for experts that return
     their input and have no matrices; `shared_gate`: the shared expert's output is multiplied by sigmoid of one more
     projection, a number per token.  Router "logits": logits + a stored bias, the `top` largest are chosen, weights = softmax
-    over the chosen ones alone.  `activation` "silu": experts with a gate, W_down (silu(W_gate h) * W_up h); "gelu": without,
-    W_down gelu(W_up h) with the erf form (the shared expert alike)."""
+    over the chosen ones alone.  Router "sigmoid": scores sigmoid(logit), chosen by score + a stored correction among the members of
+    the `group_keep` best groups (a group is as good as the sum of its two largest choice scores), weights = weight_scale x the
+    scores themselves.  `activation` "silu": experts with a gate, W_down (silu(W_gate h) * W_up h); "gelu": without,
+    W_down gelu(W_up h) with the erf form; "relu2": W_down max(W_up h, 0)^2 (the shared expert alike)."""
     experts: int
     top: int
     ff: int
@@ -620,14 +710,15 @@ class MoESpec:
     renorm: bool = True
     shared_gate: bool = False
     activation: str = "silu"
+    weight_scale: float = 1.0
 
     kind = "moe"
 
     @property
     def shared_slot(self) -> bool:
-        """A shared expert without a gate of its own that is no wider than the experts rides in their stack (padded with zero
-        rows) as one more matrix that every token takes with weight 1."""
-        return self.router == "logits" and 0 < self.shared_ff <= self.ff
+        """A shared expert no wider than the experts rides in their stack (padded with zero rows) as one more matrix that every
+        token takes, with weight 1 (router "logits", no gate) or with its gate's sigmoid (router "sigmoid")."""
+        return self.router in ("logits", "sigmoid") and 0 < self.shared_ff <= self.ff
 
     @property
     def slots(self) -> int:
@@ -643,7 +734,7 @@ class MoESpec:
 @dataclass(frozen=True)
 class LayerSpec:
     mixer: ("AttentionMixerSpec | LatentMixerSpec | LinearMixerSpec | GatedLinearMixerSpec | DeltaMixerSpec | MatrixLSTMSpec | "
-            "ParallelMixerSpec")
+            "GLAMixerSpec | ParallelMixerSpec")
     mlp: "MoESpec | DenseSpec | None"
 
 
@@ -668,6 +759,7 @@ class LayeredConfig:
     tied_head: bool = False            # the logits are products with the embedding table
     residual_mult: float = 1.0         # pre_norm blocks: factor on every sublayer's result before it joins the residual
     conv_taps: int = 0                 # > 0: h <- h + causal convolution over `conv_taps` positions in front of every sublayer
+    embed_scale: float = 1.0           # constant factor on the embedding rows
     embed_norm: bool = False           # the model's norm on the embedding output
     layer_scale: bool = False          # per-channel factors on the mixer's and the feed-forward's result
     side_dim: int = 0                  # > 0: a per-layer token input of this size after every layer
@@ -960,9 +1052,84 @@ def _vosolorn_config(d: dict) -> LayeredConfig:
                          block="post_norm", norm="rmsnorm", embed_norm=True, layer_scale=True, tied_head=True)
 
 
+def _goluzen_config(d: dict) -> LayeredConfig:
+    """Goluzen: pre-norm blocks (RMS norms whose weights are stored around zero) of three mixers -- "attention" (biases, rotation in
+    halves with linear position scaling, unit-norm q / k behind it, tanh cap, a sliding window with kept first positions, a learned
+    sink), "latent_attention" (queries projected directly, YaRN-scaled rotation in pairs, a sliding window, a gate per element; a
+    layer may read an earlier one's latent) and "gla" (gated linear attention with a decay per key channel) -- and two
+    feed-forwards without gates (gelu, or squared-ReLU experts behind a sigmoid router with group limits and a gated shared
+    expert).  What the design fixes is set here; sizes and constants come from the file."""
+
+    def sizes(m, where):
+        heads, dim = int(m["heads"]), int(m["dim"])
+        kv = int(m.get("kv_heads") or heads)
+        vdim = int(m.get("vdim") or dim)
+        if heads < 1 or dim < 1 or vdim < 1 or kv < 1 or heads % kv:
+            raise ValueError(f"{where}: {heads} heads over {kv} key/value heads")
+        return heads, kv, dim, vdim
+
+    layers: list[LayerSpec] = []
+    for i, L in enumerate(d["layers"]):
+        m, kind, where = L["mixer"], L.get("type"), f"Goluzen: layer {i}"
+        heads, kv, dim, vdim = sizes(m, where)
+        mask = m.get("mask") or {}
+        window = int(mask.get("size") or 0)
+        if window < 0:
+            raise ValueError(f"{where}: window {window}")
+        if kind == "attention":
+            mixer = AttentionMixerSpec(heads=heads, kv_heads=kv, dim=dim, vdim=vdim, scale=float(m["scale"]),
+                                       softcap=float(m.get("softcap") or 0.0), window=window,
+                                       keep_first=int(mask.get("keep_first") or 0) if window > 0 else 0,     # no window: all visible
+                                       qk_norm=True, norm_weight=False, out_gate=False, distance_bias=False, sink="learned",
+                                       rot=_rotary(m.get("rot"), dim, where), qkv_bias=True)
+        elif kind == "latent_attention":
+            rot = m.get("rot") or {}
+            sc = rot.get("scaling")
+            rot_dim = int(m["rot_dim"])
+            src = -1 if m.get("kv_from") is None else int(m["kv_from"])
+            mixer = LatentMixerSpec(heads=heads, dim=dim, rot_dim=rot_dim, vdim=vdim, kv_rank=int(m["kv_rank"]), q_rank=0,
+                                    scale=float(m["scale"]), rot_dims=int(rot.get("dims", rot_dim)), rot_base=float(rot.get("base", 10000.0)),
+                                    sink="none", gate_per_head=False, window=window, kv_from=src,
+                                    yarn=YarnSpec(float(sc["factor"]), float(sc["original"]), float(sc["fast"]), float(sc["slow"])) if sc else None)
+            if mixer.rot_dims % 2 or mixer.rot_dims > rot_dim:
+                raise ValueError(f"{where}: {mixer.rot_dims} rotated dimensions in a part of {rot_dim}")
+            if src >= 0:
+                own = layers[src].mixer if src < i else None
+                if own is None or own.kind != "latent_attention" or own.kv_from >= 0:
+                    raise ValueError(f"{where}: no latent of its own in layer {src} to read")
+                if (own.kv_rank, own.rot_dim, own.inv_freq(), own.rot_mult) != (mixer.kv_rank, rot_dim, mixer.inv_freq(), mixer.rot_mult):
+                    raise ValueError(f"{where}: latent size or rotation differ from layer {src}'s")
+        elif kind == "gla":
+            mixer = GLAMixerSpec(heads=heads, dim=dim, vdim=vdim, tau=float(m["tau"]))
+            if mixer.tau <= 0:
+                raise ValueError(f"{where}: tau {mixer.tau}")
+        else:
+            raise ValueError(f"{where} has unknown type {kind!r}")
+        mlp = None
+        f = L.get("mlp")
+        if f:
+            if f.get("kind") == "dense":
+                mlp = DenseSpec(ff=int(f["ff"]), activation="gelu_tanh_up")
+            elif f.get("kind") == "moe":
+                r, sh = f["router"], f.get("shared") or {}
+                g = r.get("groups") or {}
+                mlp = MoESpec(experts=int(r["experts"]), top=int(r["top"]), ff=int(f["expert"]["ff"]), group_count=int(g.get("count") or 1),
+                              group_keep=int(g.get("keep") or 1), shared_ff=int(sh.get("ff") or 0), router="sigmoid", renorm=False,
+                              shared_gate=bool(sh.get("ff")), activation="relu2", weight_scale=float(r.get("scale", 1.0)))
+                per = mlp.experts // mlp.group_count
+                if mlp.experts % mlp.group_count or not 1 <= mlp.top <= min(mlp.experts, per * mlp.group_keep):
+                    raise ValueError(f"{where}: top {mlp.top} of {mlp.experts} experts in {mlp.group_count} groups, {mlp.group_keep} kept")
+            else:
+                raise ValueError(f"{where} has unknown feed-forward kind {f.get('kind')!r}")
+        layers.append(LayerSpec(mixer, mlp))
+    return LayeredConfig(architecture="Goluzen", vocab_size=int(d["vocab"]), hidden_size=int(d["width"]), layers=layers,
+                         norm_eps=float((d.get("norm") or {}).get("eps", 1e-6)), block="pre_norm", norm="rmsnorm_1p",
+                         embed_scale=float((d.get("embedding") or {}).get("scale", 1.0)))
+
+
 # config.json "architecture" -> parser (the model registry of the layered families)
 LAYERED_ARCHITECTURES = {"dolurax": _dolurax_config, "turutar": _turutar_config, "rezulorn": _rezulorn_config,
-                         "sumitar": _sumitar_config, "vosolorn": _vosolorn_config}
+                         "sumitar": _sumitar_config, "vosolorn": _vosolorn_config, "goluzen": _goluzen_config}
 
 
 def layered_config_from_json(d: dict) -> LayeredConfig | None:
@@ -973,5 +1140,5 @@ def layered_config_from_json(d: dict) -> LayeredConfig | None:
 
 __all__ = ["ModelSpec", "TransformerConfig", "GPT2Config", "LlamaConfig", "Qwen3Config", "GPT2_SPEC", "LLAMA_SPEC",
            "QWEN2_SPEC", "QWEN3_SPEC", "QWEN3_MOE_SPEC", "MIXTRAL_SPEC", "MODEL_SPECS", "detect_model_spec",
-           "named_config", "AttentionMixerSpec", "LatentMixerSpec", "RotarySpec", "LinearMixerSpec", "GatedLinearMixerSpec", "DeltaMixerSpec", "MatrixLSTMSpec", "ParallelMixerSpec", "DenseSpec", "MoESpec", "LayerSpec", "LayeredConfig",
+           "named_config", "AttentionMixerSpec", "LatentMixerSpec", "RotarySpec", "YarnSpec", "LinearMixerSpec", "GLAMixerSpec", "GatedLinearMixerSpec", "DeltaMixerSpec", "MatrixLSTMSpec", "ParallelMixerSpec", "DenseSpec", "MoESpec", "LayerSpec", "LayeredConfig",
            "LAYERED_ARCHITECTURES", "layered_config_from_json"]

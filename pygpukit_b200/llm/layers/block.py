@@ -237,6 +237,74 @@ class PreNormBlock:
         return n
 
 
+class PreNormSeamBlock:
+    """Pre-norm block with RMS norms and nothing between norm and sublayer: x += mixer(norm1(x)), then x += ff(norm2(x)).  A sublayer
+    leaves its result as rows of its own (experts: as the rows still to be summed), and the seam behind it is ONE launch
+    (pgk_rms_add_norm_f32): the weighted sum of the chosen experts with the gated shared expert, the residual add, and the norm in
+    front of the next sublayer -- the feed-forward's, or the next block's first one.  Per-sequence state of the block in the cache
+    manager: whatever the mixer keeps."""
+
+    def __init__(self, norm1, mixer, norm2=None, mlp=None):
+        self.norm1, self.mixer, self.norm2, self.mlp = norm1, mixer, norm2, mlp
+        if (mlp is None) != (norm2 is None):
+            raise ValueError("PreNormSeamBlock: a feed-forward comes with its norm")
+        if any(n is not None and n.kind != "rmsnorm" for n in (norm1, norm2)):
+            raise ValueError("PreNormSeamBlock: the seam takes RMS norms")
+
+    @property
+    def norm(self):
+        """the norm in front of the block: the block before may write its rows"""
+        return self.norm1
+
+    @property
+    def state_shapes(self) -> tuple:
+        return tuple(self.mixer.spec.state_shapes)
+
+    def forward(self, ctx, x: GPUArray, cache_index: int | None = None, add_ptr: int | None = None, normed: bool = False,
+                next_norm=None, next_add_ptr: int | None = None) -> bool:
+        """normed: ctx.buf.h already holds norm1(x) (the block before wrote it).  next_norm: the first norm of the block that
+        runs next; returns True when this block has written that block's normed rows."""
+        if add_ptr is not None or next_add_ptr is not None:
+            raise ValueError("PreNormSeamBlock: no loop passes in this block form")
+        h, y = ctx.buf.h, ctx.buf.y
+        if next_norm is not None and next_norm.kind != "rmsnorm":
+            next_norm = None
+        if not normed:
+            self._seam(ctx, {}, x, self.norm1)
+        if self.state_shapes:
+            self.mixer.forward(ctx, h, y, cache_index, state=ctx.cache.state[cache_index])
+        else:
+            self.mixer.forward(ctx, h, y, cache_index)
+        rows = {"y": y.device_ptr}
+        if self.mlp is None:
+            return self._seam(ctx, rows, x, next_norm)
+        self._seam(ctx, rows, x, self.norm2)
+        if hasattr(self.mlp, "forward_pending"):
+            return self._seam(ctx, self.mlp.forward_pending(ctx, h, y), x, next_norm)
+        self.mlp.forward(ctx, h.device_ptr, y.device_ptr)
+        return self._seam(ctx, rows, x, next_norm)
+
+    @staticmethod
+    def _seam(ctx, p: dict, x: GPUArray, nxt) -> bool:
+        """x += the pending result ({}: nothing); h = nxt(x) when there is one (returns whether)"""
+        from ..._lib import api
+        from ...core.stream import current_stream_handle as _st
+        if p.get("self_rows") is not None and p.get("mat") is not None:
+            raise ValueError("PreNormSeamBlock: experts without matrices are not summed by this seam")
+        api.rms_add_norm_f32(p.get("y"), p.get("parts"), p.get("inv"), p.get("w"), p.get("top", 0), p.get("shared"), p.get("gate"),
+                             p.get("ldg", 0), p.get("gate_off", 0), x.device_ptr, nxt.weight.device_ptr if nxt is not None else None,
+                             nxt.offset if nxt is not None else 0.0, nxt.eps if nxt is not None else 0.0,
+                             ctx.buf.h.device_ptr if nxt is not None else None, ctx.T, x.shape[1], _st())
+        return nxt is not None
+
+    @property
+    def weight_bytes(self) -> int:
+        n = self.mixer.weight_bytes + self.norm1.nbytes
+        if self.mlp is not None:
+            n += self.mlp.weight_bytes + self.norm2.nbytes
+        return n
+
+
 class SandwichBlock:
     """Block of the token-major models with a norm before AND after each sublayer: x += norm1b(mixer(norm1(x))), then
     x += norm2b(ff(norm2(x))).  The norms are `RowNorm`s of any kind.  With dynamic-tanh norms the seam behind a sublayer is
@@ -323,4 +391,4 @@ class SandwichBlock:
         return n
 
 
-__all__ = ["TransformerBlock", "PostNormBlock", "ParallelBlock", "PreNormBlock", "SandwichBlock"]
+__all__ = ["TransformerBlock", "PostNormBlock", "ParallelBlock", "PreNormBlock", "PreNormSeamBlock", "SandwichBlock"]

@@ -6,8 +6,8 @@ interleaved (gate_j, up_j) pairs, and the down projection.
   activation "gelu_tanh":      gelu(g) * u, the tanh form
   activation "clamped_swish":  g <- min(g, limit), u <- clamp(u, -limit, limit), g * sigmoid(alpha g) * (u + 1)
 
-`SquaredReluRows` is the feed-forward without a gate, W_down max(W_up h, 0)^2, the activation again in the first product's
-epilogue.
+`ActivatedRows` is the feed-forward without a gate, the activation again in the first product's epilogue: "relu2",
+W_down max(W_up h, 0)^2, or "gelu_tanh_up", W_down gelu(W_up h) with the tanh form.
 
 `forward(..., out_scale=ptr)` adds `out_scale * result` to `out` in the down projection's epilogue (layer scale and
 residual add of a parallel block); without it the result is stored.
@@ -43,12 +43,14 @@ class GatedDenseRows:
             self.down.forward_seq(act.device_ptr, sp.ff, T, out_ptr, self.down.out_features, epilogue=4, col_scale=out_scale)
 
 
-class SquaredReluRows:
+class ActivatedRows:
+    EPILOGUES = {"relu2": 6, "gelu_tanh_up": 9}
+
     def __init__(self, spec: DenseSpec, up: LinearRows, down: LinearRows):
-        if spec.activation != "relu2":
-            raise ValueError(f"SquaredReluRows: activation {spec.activation!r}")
+        if spec.activation not in self.EPILOGUES:
+            raise ValueError(f"{type(self).__name__}: activation {spec.activation!r}")
         if up.out_features != spec.ff or down.in_features != spec.ff:
-            raise ValueError("SquaredReluRows: matrices do not match the feed-forward size")
+            raise ValueError(f"{type(self).__name__}: matrices do not match the feed-forward size")
         self.spec, self.up, self.down = spec, up, down
 
     @property
@@ -58,11 +60,15 @@ class SquaredReluRows:
     def forward(self, ctx, h_ptr: int, out_ptr: int, out_scale: int | None = None) -> None:
         sp, T = self.spec, ctx.T
         W, act = self.up.in_features, ctx.buf.shared_act
-        self.up.forward_seq(h_ptr, W, T, act.device_ptr, sp.ff, epilogue=6)
+        self.up.forward_seq(h_ptr, W, T, act.device_ptr, sp.ff, epilogue=self.EPILOGUES[sp.activation])
         if out_scale is None:
             self.down.forward_seq(act.device_ptr, sp.ff, T, out_ptr, self.down.out_features, epilogue=0)
         else:
             self.down.forward_seq(act.device_ptr, sp.ff, T, out_ptr, self.down.out_features, epilogue=4, col_scale=out_scale)
+
+
+class SquaredReluRows(ActivatedRows):
+    EPILOGUES = {"relu2": 6}
 
 
 class PolyNormRows:
@@ -99,4 +105,4 @@ class PolyNormRows:
         self.forward(ctx, x.device_ptr, out.device_ptr)
 
 
-__all__ = ["GatedDenseRows", "SquaredReluRows", "PolyNormRows"]
+__all__ = ["GatedDenseRows", "ActivatedRows", "SquaredReluRows", "PolyNormRows"]

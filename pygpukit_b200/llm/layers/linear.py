@@ -247,9 +247,9 @@ class LinearRows:
     [E, N, K] of expert matrices) in bfloat16 or float32, float32 accumulation and output.  Many rows run as tiled
     GEMMs (tensor cores for bfloat16 weights), up to eight rows through the streaming few-row kernel.  epilogue:
     0 plain, 1 gate/up pairs -> silu(gate) * up (rows of W interleaved by `interleave_gate_up`), 2 scale + tanh cap,
-    7 gate/up pairs -> gelu_tanh(gate) * up, 8 gelu (erf form) of the product;
+    6 squared ReLU, 7 gate/up pairs -> gelu_tanh(gate) * up, 8 / 9 gelu (erf / tanh form) of the product;
     `forward_seq` adds 3 clamped gate/up pairs, 4 scaled accumulation into the output, 5 gelu * gathered table entry,
-    and batches of per-head products."""
+    10 product * sigmoid(gate row's element), and batches of per-head products."""
 
     FEW = 8
     FEW_SMEM_FLOATS = 40960          # 160 KB of activations per block
@@ -290,7 +290,8 @@ class LinearRows:
                     batch: int = 1, a_batch: int = 0, c_batch: int = 0) -> None:
         """The general product (pgk_gemm_seq_f32).  epilogue 3: clamped gate/up pairs (p0 = alpha, p1 = limit); 4: out +=
         col_scale * product (col_scale: device pointer of [N] floats); 5: gelu_tanh(product) * aux entry, aux = (table
-        pointer, dtype code, row-index pointer, row stride, column offset).  batch > 1: the weight is a stack [batch, N, K]
+        pointer, dtype code, row-index pointer, row stride, column offset); 10: product * sigmoid(aux element of the same row and
+        column), aux the same tuple without row indices (batches: the gate's columns lie c_batch apart like the output's).  batch > 1: the weight is a stack [batch, N, K]
         and product b reads x columns from b * a_batch and writes out columns from b * c_batch."""
         N, K = self.out_features, self.in_features
         epi = self.epilogue if epilogue is None else epilogue

@@ -88,28 +88,34 @@ class GroupedRouterMoE:
 
 class BiasedRouterMoE:
     """Mixture of experts whose router adds a stored correction to the scores when it CHOOSES (the weights are the scores
-    themselves, renormalised or not), whose last `identity` router outputs stand for experts that return their input, and
+    themselves, renormalised, scaled or not; softmax scores, or with spec.router "sigmoid" sigmoid ones with group limits), whose last `identity` router outputs stand for experts that return their input, and
     whose shared expert is multiplied by sigmoid of one more projection (a number per token).  The router matrix, float32 in
     both modes, carries the shared expert's gate as its last row, so that one product gives both.  Experts and row lists as in
     `GroupedRouterMoE` (rows of experts without matrices sort behind the others and no product touches them; among few rows
     they are skipped by their matrix number -1).  `forward_rows` leaves the layer's result in `out`:
 
-      pgk_moe_route_biased      scores, choice, weights, row lists
+      pgk_moe_route_biased / pgk_moe_route_sigmoid   scores, choice, weights, row lists
       pgk_moe_combine_rows_f32  weighted sum of the chosen experts' rows (or the token's own row) + gated shared expert
     """
 
     def __init__(self, spec: MoESpec, router: GPUArray, correction: "GPUArray | None", gate_up: "LinearRows | None",
                  down: "LinearRows | None", shared_gate_up: LinearRows | None = None, shared_down: LinearRows | None = None):
-        """router: [routes (+ 1 with a gated shared expert), W] float32."""
+        """router: [routes (+ 1 with a gated shared expert), W] float32.  Experts without gates put the up matrices in `gate_up`
+        with their activation's epilogue; a shared expert that rides in the stack (spec.shared_slot) is its last matrix."""
         self.spec, self.router, self.correction = spec, LinearRows(router), correction
         self.gate_up, self.down = gate_up, down
         self.shared_gate_up, self.shared_down = shared_gate_up, shared_down
         self.z_cols = spec.routes + (1 if spec.shared_gate else 0)
         if self.router.out_features != self.z_cols:
             raise ValueError(f"BiasedRouterMoE: the router has {self.router.out_features} rows, the spec needs {self.z_cols}")
-        if spec.experts > 0 and (gate_up is None or gate_up.groups != spec.experts or down.groups != spec.experts):
+        self.stack = spec.experts + (1 if spec.shared_slot else 0)
+        if spec.router not in ("biased", "sigmoid") or (spec.router == "sigmoid" and (spec.identity or spec.renorm)):
+            raise ValueError(f"BiasedRouterMoE: router {spec.router!r}, {spec.identity} experts without matrices")
+        if spec.experts > 0 and (gate_up is None or gate_up.groups != self.stack or down.groups != self.stack):
             raise ValueError("BiasedRouterMoE: expert stacks do not match the router")
-        if bool(spec.shared_ff) != (shared_gate_up is not None) or (spec.shared_gate and not spec.shared_ff):
+        if spec.shared_slot and not spec.shared_gate:
+            raise ValueError("BiasedRouterMoE: a shared expert in the stack is weighed by its gate")
+        if (bool(spec.shared_ff) and not spec.shared_slot) != (shared_gate_up is not None) or (spec.shared_gate and not spec.shared_ff):
             raise ValueError("BiasedRouterMoE: the shared expert and the spec do not agree")
 
     @property
@@ -130,21 +136,28 @@ class BiasedRouterMoE:
         """Everything but the weighted sum, for a block that folds the sum into its own seam launch: the description of the
         rows to be summed ("experts")."""
         sp, T, b = self.spec, ctx.T, ctx.buf
-        W, top, ff, R = self.router.in_features, sp.top, sp.ff, sp.routes
+        W, top, ff, R = self.router.in_features, sp.slots, sp.ff, sp.routes
         few = T <= LinearRows.FEW
         self.router.forward(x.device_ptr, W, T, b.moe_z.device_ptr, self.z_cols)          # float32 logits [T, routes (+ 1)]
-        api.moe_route_biased(b.moe_z.device_ptr, self.z_cols, T, R, sp.experts, top,
-                             self.correction.device_ptr if self.correction is not None else None, 1 if sp.renorm else 0,
-                             b.moe_idx.device_ptr, b.moe_mat.device_ptr, b.moe_w.device_ptr,
-                             None if few else b.moe_rank.device_ptr, None if few else b.moe_counts.device_ptr, _st())
+        corr = self.correction.device_ptr if self.correction is not None else None
+        rank, counts = (None, None) if few else (b.moe_rank.device_ptr, b.moe_counts.device_ptr)
+        mat = b.moe_mat                                  # the matrix of every (token, slot) row, -1: none
+        if sp.router == "sigmoid":
+            mat = b.moe_idx                              # every choice has one
+            api.moe_route_sigmoid(b.moe_z.device_ptr, self.z_cols, T, sp.experts, sp.top, corr, sp.group_count, sp.group_keep,
+                                  sp.weight_scale, sp.experts if sp.shared_slot else -1, b.moe_idx.device_ptr, b.moe_w.device_ptr,
+                                  rank, counts, _st())
+        else:
+            api.moe_route_biased(b.moe_z.device_ptr, self.z_cols, T, R, sp.experts, top, corr, 1 if sp.renorm else 0,
+                                 b.moe_idx.device_ptr, b.moe_mat.device_ptr, b.moe_w.device_ptr, rank, counts, _st())
         if few:
             slot_tok, inv = ctx.slot_rows(top)
             if sp.experts > 0:
-                self.gate_up.forward_per_row(x.device_ptr, W, T * top, b.moe_act.device_ptr, ff, slot_tok, b.moe_mat.device_ptr)
-                self.down.forward_per_row(b.moe_act.device_ptr, ff, T * top, b.moe_parts.device_ptr, W, None, b.moe_mat.device_ptr)
+                self.gate_up.forward_per_row(x.device_ptr, W, T * top, b.moe_act.device_ptr, ff, slot_tok, mat.device_ptr)
+                self.down.forward_per_row(b.moe_act.device_ptr, ff, T * top, b.moe_parts.device_ptr, W, None, mat.device_ptr)
         else:
             api.moe_row_lists(b.moe_counts.device_ptr, b.moe_off.device_ptr, b.moe_idx.device_ptr, b.moe_rank.device_ptr,
-                              b.moe_perm.device_ptr, b.moe_inv.device_ptr, R, T, top, _st())
+                              b.moe_perm.device_ptr, b.moe_inv.device_ptr, max(R, self.stack), T, top, _st())
             if sp.experts > 0:
                 self.gate_up.forward_grouped(x.device_ptr, W, b.moe_act.device_ptr, ff, b.moe_perm.device_ptr,
                                              b.moe_off.device_ptr, T)
@@ -156,8 +169,9 @@ class BiasedRouterMoE:
             self.shared_gate_up.forward(x.device_ptr, W, T, b.shared_act.device_ptr, fs)
             self.shared_down.forward(b.shared_act.device_ptr, fs, T, b.y2.device_ptr, W)
             shared = b.y2.device_ptr
-        return {"mode": "experts", "parts": b.moe_parts.device_ptr, "inv": inv, "mat": b.moe_mat.device_ptr, "w": b.moe_w.device_ptr,
-                "top": top, "self_rows": x.device_ptr, "shared": shared, "gate": b.moe_z.device_ptr if sp.shared_gate else None,
+        return {"mode": "experts", "parts": b.moe_parts.device_ptr, "inv": inv, "mat": mat.device_ptr if sp.router == "biased" else None,
+                "w": b.moe_w.device_ptr, "top": top, "self_rows": x.device_ptr, "shared": shared,
+                "gate": b.moe_z.device_ptr if sp.shared_gate else None,
                 "ldg": self.z_cols, "gate_off": R}
 
 

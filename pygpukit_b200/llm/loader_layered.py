@@ -37,9 +37,17 @@ l<i>.mix.{q,k,v,o}, .q.norm, .k.norm [dim]; "mlstm" l<i>.mix.{q,k,v,g,o}, .norm 
 .f.b; dense feed-forward l<i>.mlp.{gate,up,down}; experts l<i>.mlp.e<j>.{up,down}, .router [experts, width] with .router.b,
 .shared.{up,down}.  An mLSTM mixer's projections are one matrix [q | k | v | g | i | f]; a layer scale multiplies the weight of the
 norm in front of it; a shared expert no wider than the others is the last matrix of their stack.
+
+Goluzen tensor names: embed, final.norm, head; per layer l<i>.norm1, norm2; "attention" l<i>.mix.{q,k,v} with biases .q.b / .k.b /
+.v.b, .sink [heads], .o; "latent_attention" l<i>.mix.{q,g,uk,uv,o} and, without kv_from, .dkv, .dkv.norm; "gla"
+l<i>.mix.{q,k,v,g,o}, .a1 [inner, width], .a2 [heads x dim, inner], .a2.b, .norm [vdim]; dense feed-forward l<i>.mlp.{up,down};
+experts l<i>.mlp.e<j>.{up,down}, .router, .correction, .shared.{up,down,sg}.  Fused projections [q | k | v], [q | dkv | g] and
+[q | k | v | g | a1]; uk and uv as Turutar's; a2 stored transposed; the router matrix carries the shared expert's gate row as its
+last row; a shared expert no wider than the others is the last matrix of their stack.  The inner size of the decays is read from a1.
 """
 from __future__ import annotations
 
+import dataclasses
 import json
 import os
 
@@ -49,9 +57,10 @@ from ..core.array import GPUArray
 from ..core.dtypes import bf16_bits_to_f32, f32_to_bf16_bits
 from ..core.factory import from_numpy
 from .config import LayeredConfig, layered_config_from_json
-from .layers.block import ParallelBlock, PostNormBlock, PreNormBlock, SandwichBlock
-from .layers.dense_rows import GatedDenseRows, PolyNormRows, SquaredReluRows
+from .layers.block import ParallelBlock, PostNormBlock, PreNormBlock, PreNormSeamBlock, SandwichBlock
+from .layers.dense_rows import ActivatedRows, GatedDenseRows, PolyNormRows, SquaredReluRows
 from .layers.gated_recurrent import DeltaRuleMixer, GatedLinearMixer
+from .layers.gla import GLAMixer
 from .layers.linear_attention import LinearAttentionMixer, ParallelMixer
 from .layers.latent_attention import LatentAttentionMixer
 from .layers.linear import LinearRows, interleave_gate_up
@@ -356,20 +365,12 @@ def _build_vosolorn(config: LayeredConfig, t: _Tensors, dtype: str) -> LayeredCa
                 gu = interleave_gate_up(t.f32(q + "gate", (f.ff, W)), t.f32(q + "up", (f.ff, W)))
                 mlp = GatedDenseRows(f, LinearRows(_matrix(gu, dtype)), LinearRows(_matrix(t.f32(q + "down", (W, f.ff)), dtype)))
             else:
-                up = [t.f32(f"{q}e{e}.up", (f.ff, W)) for e in range(f.experts)]
-                dn = [t.f32(f"{q}e{e}.down", (W, f.ff)) for e in range(f.experts)]
-                sup = sdn = None
-                if f.shared_ff:
-                    su, sd = t.f32(q + "shared.up", (f.shared_ff, W)), t.f32(q + "shared.down", (W, f.shared_ff))
-                    if f.shared_slot:
-                        pad = f.ff - f.shared_ff
-                        up.append(np.pad(su, ((0, pad), (0, 0))))
-                        dn.append(np.pad(sd, ((0, 0), (0, pad))))
-                    else:
-                        sup, sdn = LinearRows(_matrix(su, dtype), epilogue=8), LinearRows(_matrix(sd, dtype))
+                up, dn, sup, sdn = _stack_experts(t, q, f, W)
+                if sup is not None:
+                    sup, sdn = LinearRows(_matrix(sup, dtype), epilogue=8), LinearRows(_matrix(sdn, dtype))
                 # the router stays float32 in both modes: its logits come from the unrounded residual stream
                 mlp = GroupedRouterMoE(f, _matrix(t.f32(q + "router", (f.experts, W)), "float32"),
-                                       LinearRows(_matrix(np.stack(up), dtype), epilogue=8), LinearRows(_matrix(np.stack(dn), dtype)),
+                                       LinearRows(_matrix(up, dtype), epilogue=8), LinearRows(_matrix(dn, dtype)),
                                        sup, sdn, router_bias=_vector(t.f32(q + "router.b", (f.experts,))))
         blocks.append(PostNormBlock(mixer, norm(p + "norm1", p + "ls1"), mlp, norm2, eps))
     embed = _matrix(t.f32("embed", (V, W)), dtype)
@@ -377,9 +378,85 @@ def _build_vosolorn(config: LayeredConfig, t: _Tensors, dtype: str) -> LayeredCa
     return LayeredCausalModel(config, embed, blocks, norm("final.norm"), head, dtype, embed_norm=norm("embed.norm"))
 
 
+def _stack_experts(t: _Tensors, q: str, f, W: int) -> tuple:
+    """(up stack, down stack, shared up or None, shared down or None) of experts without gates; a shared expert that rides in the
+    stack is its last matrix, padded with zero rows / columns"""
+    up = [t.f32(f"{q}e{e}.up", (f.ff, W)) for e in range(f.experts)]
+    dn = [t.f32(f"{q}e{e}.down", (W, f.ff)) for e in range(f.experts)]
+    sup = sdn = None
+    if f.shared_ff:
+        sup, sdn = t.f32(q + "shared.up", (f.shared_ff, W)), t.f32(q + "shared.down", (W, f.shared_ff))
+        if f.shared_slot:
+            pad = f.ff - f.shared_ff
+            up.append(np.pad(sup, ((0, pad), (0, 0))))
+            dn.append(np.pad(sdn, ((0, 0), (0, pad))))
+            sup = sdn = None
+    return np.stack(up), np.stack(dn), sup, sdn
+
+
+def _build_goluzen(config: LayeredConfig, t: _Tensors, dtype: str) -> LayeredCausalModel:
+    W, V, eps = config.hidden_size, config.vocab_size, config.norm_eps
+
+    def norm(name):                           # weights stored around zero
+        return RowNorm("rmsnorm", _vector(t.f32(name, (W,))), None, eps, offset=1.0)
+
+    def rows(a):
+        return LinearRows(_matrix(a, dtype))
+
+    layers = []                               # the inner size of a decay is known from its matrices alone
+    for i, L in enumerate(config.layers):
+        m = L.mixer
+        if m.kind == "gla":
+            m = dataclasses.replace(m, gate_rank=int(t.f32(f"l{i}.mix.a1").shape[0]))
+        layers.append(dataclasses.replace(L, mixer=m))
+    config = dataclasses.replace(config, layers=layers)
+    blocks = []
+    for i, L in enumerate(config.layers):
+        p, m = f"l{i}.", L.mixer
+        mp = p + "mix."
+        H, D, Dv = m.heads, m.dim, m.vdim
+        o_proj = rows(t.f32(mp + "o", (W, H * Dv)))
+        if m.kind == "attention":
+            qd, kd, vd = H * D, m.kv_heads * D, m.kv_heads * Dv
+            fused = np.concatenate([t.f32(mp + "q", (qd, W)), t.f32(mp + "k", (kd, W)), t.f32(mp + "v", (vd, W))])
+            mixer = PagedAttentionMixer(m, i, rows(fused), o_proj, None, None, eps, q_bias=_vector(t.f32(mp + "q.b", (qd,))),
+                                        k_bias=_vector(t.f32(mp + "k.b", (kd,))), v_bias=_vector(t.f32(mp + "v.b", (vd,))),
+                                        sinks=_vector(t.f32(mp + "sink", (H,))))
+        elif m.kind == "latent_attention":
+            R, own = m.kv_rank, m.kv_from < 0
+            parts = [t.f32(mp + "q", (H * (D + m.rot_dim), W))]
+            if own:
+                parts.append(t.f32(mp + "dkv", (R + m.rot_dim, W)))
+            parts.append(t.f32(mp + "g", (H * Dv, W)))
+            uk = t.f32(mp + "uk", (H * D, R)).reshape(H, D, R).transpose(0, 2, 1)
+            uv = t.f32(mp + "uv", (H * Dv, R)).reshape(H, Dv, R)
+            mixer = LatentAttentionMixer(m, i, rows(np.concatenate(parts)), None, rows(uk), rows(uv), o_proj, None,
+                                         _vector(t.f32(mp + "dkv.norm", (R,))) if own else None, eps)
+        else:
+            fused = np.concatenate([t.f32(mp + "q", (H * D, W)), t.f32(mp + "k", (H * D, W)), t.f32(mp + "v", (H * Dv, W)),
+                                    t.f32(mp + "g", (H * Dv, W)), t.f32(mp + "a1", (m.gate_rank, W))])
+            mixer = GLAMixer(m, i, rows(fused), o_proj, _vector(t.f32(mp + "a2", (H * D, m.gate_rank)).T), _vector(t.f32(mp + "a2.b", (H * D,))),
+                             _vector(np.tile(t.f32(mp + "norm", (Dv,)), H)), eps)
+        mlp, f, q = None, L.mlp, p + "mlp."
+        if f is not None and f.kind == "dense":
+            mlp = ActivatedRows(f, rows(t.f32(q + "up", (f.ff, W))), rows(t.f32(q + "down", (W, f.ff))))
+        elif f is not None:
+            up, dn, sup, sdn = _stack_experts(t, q, f, W)
+            router = [t.f32(q + "router", (f.experts, W))]
+            if f.shared_gate:
+                router.append(t.f32(q + "shared.sg", (1, W)))
+            # the router (and the gate row it carries) stays float32 in both modes
+            mlp = BiasedRouterMoE(f, _matrix(np.concatenate(router), "float32"), _vector(t.f32(q + "correction", (f.experts,))),
+                                  LinearRows(_matrix(up, dtype), epilogue=6), rows(dn),
+                                  LinearRows(_matrix(sup, dtype), epilogue=6) if sup is not None else None,
+                                  rows(sdn) if sdn is not None else None)
+        blocks.append(PreNormSeamBlock(norm(p + "norm1"), mixer, norm(p + "norm2") if mlp is not None else None, mlp))
+    return LayeredCausalModel(config, _matrix(t.f32("embed", (V, W)), dtype), blocks, norm("final.norm"), rows(t.f32("head", (V, W))), dtype)
+
+
 # architecture (lower case) -> builder of its blocks from the checkpoint's tensors
 _BUILDERS = {"dolurax": _build_dolurax, "turutar": _build_turutar, "rezulorn": _build_rezulorn, "sumitar": _build_sumitar,
-             "vosolorn": _build_vosolorn}
+             "vosolorn": _build_vosolorn, "goluzen": _build_goluzen}
 
 
 def load_layered_model(model_path: str, dtype: str = "bfloat16", config: dict | None = None) -> LayeredCausalModel:

@@ -132,8 +132,12 @@ class LayeredCausalModel:
             final_norm = RowNorm("layernorm", final_norm[0], final_norm[1], config.norm_eps)
         self.final_norm, self.lm_head, self.dtype = final_norm, lm_head, dtype
         self.embed_norm = embed_norm
+        if config.embed_scale != 1.0 and embed_norm is not None:
+            raise ValueError("LayeredCausalModel: a factor on the embedding rows is built for models without an embedding norm")
         if bool(config.embed_norm) != (embed_norm is not None):
             raise ValueError("LayeredCausalModel: the config and the embedding norm do not agree")
+        if len(config.layer_runs()) != len(config.layers) and any(getattr(L.mixer, "kv_from", -1) >= 0 for L in config.layers):
+            raise ValueError("LayeredCausalModel: a layer that reads another one's cache names it by layer, not by loop pass")
         self.runs = config.layer_runs()                 # (layer, add the embedding output first); index = cache
         self.trace_hook = None                          # debugging aid: called with (run index, residual rows array)
         self.embed_dt = 2 if embed_tokens.dtype.name == "bfloat16" else 0
@@ -187,7 +191,8 @@ class LayeredCausalModel:
             api.embed_norm_rows_f32(self.embed_tokens.device_ptr, self.embed_dt, ctx.tok_ptr, en.weight.device_ptr, en.offset,
                                     en.eps, x.device_ptr, b.x0.device_ptr if b.x0 is not None else None, T, W, V, _st())
         else:
-            api.embed_rows_f32(self.embed_tokens.device_ptr, self.embed_dt, ctx.tok_ptr, x.device_ptr, T, W, V, _st())
+            api.embed_rows_scaled_f32(self.embed_tokens.device_ptr, self.embed_dt, ctx.tok_ptr, cfg.embed_scale, x.device_ptr, T, W, V,
+                                      _st())
             if en is not None:
                 en.forward(x.device_ptr, x.device_ptr, T, W)
             if b.x0 is not None:

@@ -311,6 +311,8 @@ def random_layered_model(config, dtype: str = "bfloat16", seed: int = 1234, std:
 
     if config.block == "parallel":
         return _random_parallel_model(config, dtype, mat, vec)
+    if config.block == "pre_norm" and config.norm == "rmsnorm_1p":
+        return _random_pre_rms_model(config, dtype, mat, vec)
     if config.block == "pre_norm":
         return _random_pre_norm_model(config, dtype, mat, vec)
     if config.block == "sandwich":
@@ -430,6 +432,56 @@ def _random_pre_norm_model(config, dtype, mat, vec):
         blocks.append(PreNormBlock(norm(), conv(), mixer, norm2, conv2, mlp, mult))
     head = LinearRows(mat(V, W), epilogue=2, scale=config.logit_scale, cap=0.0)
     return LayeredCausalModel(config, mat(V, W), blocks, norm(), head, dtype)
+
+
+def _random_pre_rms_model(config, dtype, mat, vec):
+    """The RMS-normed pre-norm form of `random_layered_model` (windowed attention with a sink and biases, latent attention with shared
+    latents, gated linear attention, gelu feed-forward, experts behind a sigmoid router): random matrices, norms at identity, zero
+    biases, sinks and corrections; a decay's inner size that the config does not know is 16."""
+    import dataclasses
+
+    from ..core.dtypes import float32
+    from .layers.block import PreNormSeamBlock
+    from .layers.dense_rows import ActivatedRows
+    from .layers.gla import GLAMixer
+    from .layers.latent_attention import LatentAttentionMixer
+    from .layers.linear import LinearRows
+    from .layers.moe_rows import BiasedRouterMoE
+    from .layers.norm import RowNorm
+    from .layers.paged_attention import PagedAttentionMixer
+    from .models.layered import LayeredCausalModel
+    W, V, eps = config.hidden_size, config.vocab_size, config.norm_eps
+    config = dataclasses.replace(config, layers=[
+        dataclasses.replace(L, mixer=dataclasses.replace(L.mixer, gate_rank=L.mixer.gate_rank or 16)) if L.mixer.kind == "gla" else L
+        for L in config.layers])
+
+    def norm():
+        return RowNorm("rmsnorm", vec(W, 0.0), None, eps, offset=1.0)
+
+    blocks = []
+    for i, L in enumerate(config.layers):
+        m, f = L.mixer, L.mlp
+        H, D, Dv = m.heads, m.dim, m.vdim
+        proj, o_proj = LinearRows(mat(m.proj_cols, W)), LinearRows(mat(W, H * Dv))
+        if m.kind == "attention":
+            mixer = PagedAttentionMixer(m, i, proj, o_proj, None, None, eps, q_bias=vec(H * D, 0.0), k_bias=vec(m.kv_heads * D, 0.0),
+                                        v_bias=vec(m.kv_heads * Dv, 0.0), sinks=vec(H, 0.0))
+        elif m.kind == "latent_attention":
+            mixer = LatentAttentionMixer(m, i, proj, None, LinearRows(mat(H, m.kv_rank, D)), LinearRows(mat(H, Dv, m.kv_rank)), o_proj,
+                                         None, vec(m.kv_rank, 1.0) if m.kv_from < 0 else None, eps)
+        else:
+            mixer = GLAMixer(m, i, proj, o_proj, mat(m.gate_rank, H * D).astype(float32), vec(H * D, 3.0), vec(H * Dv, 1.0), eps)
+        mlp = None
+        if f is not None and f.kind == "dense":
+            mlp = ActivatedRows(f, LinearRows(mat(f.ff, W)), LinearRows(mat(W, f.ff)))
+        elif f is not None:
+            n, own = f.experts + (1 if f.shared_slot else 0), bool(f.shared_ff) and not f.shared_slot
+            mlp = BiasedRouterMoE(f, mat(f.experts + (1 if f.shared_gate else 0), W).astype(float32), vec(f.experts, 0.0),
+                                  LinearRows(mat(n, f.ff, W), epilogue=6), LinearRows(mat(n, W, f.ff)),
+                                  LinearRows(mat(f.shared_ff, W), epilogue=6) if own else None,
+                                  LinearRows(mat(W, f.shared_ff)) if own else None)
+        blocks.append(PreNormSeamBlock(norm(), mixer, norm() if mlp is not None else None, mlp))
+    return LayeredCausalModel(config, mat(V, W), blocks, norm(), LinearRows(mat(V, W)), dtype)
 
 
 def _random_sandwich_model(config, dtype, mat, vec):
