@@ -47,6 +47,11 @@ experts with a choice bias) beside a Rezulorn stack at equal sizes, the closest 
 The same for the Vosolorn design (the matrix memory of xLSTM, attention with pooled blocks before its window, gelu experts
 behind a logit router) beside a Rezulorn stack at equal sizes, the closest existing model.
 
+    python bench.py --goluzen [--goluzen-sizes g-2048,g-4096] [--steps K] [--warmup W]
+The same for the Goluzen design (gated linear attention, windowed latent attention with shared latents, attention with kept first
+positions and a sink, squared-ReLU experts behind a sigmoid router) beside a Sumitar stack and a Turutar stack at equal sizes, the two
+closest existing models (each has the like of some of its mixers).
+
     python bench.py --turutar [--turutar-sizes t-2048,t-4096] [--steps K] [--warmup W]
 The same for the Turutar design (latent + windowed attention, gated dense feed-forward, token side inputs, a looped pair of
 layers) next to a Dolurax stack of equal size, the closest existing model: same family, same cache and kernels.
@@ -116,6 +121,11 @@ def parse_args():
                          "xLSTM, attention with pooled blocks before its window, gelu experts behind a logit router) beside a "
                          "Rezulorn stack at equal sizes, one JSON line")
     ap.add_argument("--vosolorn-sizes", default="v-2048,v-4096")
+    ap.add_argument("--goluzen", action="store_true",
+                    help="instead of the default workload: prefill / decode throughput of the Goluzen design (gated linear attention, "
+                         "windowed latent attention with shared latents, squared-ReLU experts behind a sigmoid router) beside a Sumitar "
+                         "and a Turutar stack at equal sizes, one JSON line")
+    ap.add_argument("--goluzen-sizes", default="g-2048,g-4096")
     return ap.parse_args()
 
 
@@ -641,6 +651,11 @@ def run_ours(args) -> None:
 
 def main():
     args = parse_args()
+    if args.goluzen:
+        sys.path.insert(0, os.path.join(ROOT, "scripts"))
+        import bench_layered
+        print(json.dumps(bench_layered.main_goluzen(ROOT, args.goluzen_sizes.split(","), args.steps, args.warmup)))
+        return
     if args.vosolorn:
         sys.path.insert(0, os.path.join(ROOT, "scripts"))
         import bench_layered

@@ -71,6 +71,18 @@ VOSOLORN_SIZES = {
 }
 
 
+# Goluzen: pre-norm blocks; a latent layer and one that reads its latents (gelu feed-forward), a gated-linear-attention layer and a
+# windowed attention layer (squared-ReLU experts, four of sixteen and a gated shared one of the same size)
+GOLUZEN_SIZES = {
+    "g-2048": dict(width=2048, heads=16, kv_heads=4, dim=128, window=1024, keep=4, rot=64, ldim=128, lrot=64, lvdim=128, kv_rank=512,
+                   q_rank=768, lin_heads=16, lin_dim=128, lin_vdim=128, inner=16, qk_heads=4, taps=4, ff=8192, experts=16, identity=2, top=4,
+                   groups=(4, 2), eff=2048, shared_ff=2048, side=0, times=1, vocab=32768),
+    "g-4096": dict(width=4096, heads=32, kv_heads=8, dim=128, window=2048, keep=4, rot=64, ldim=128, lrot=64, lvdim=128, kv_rank=512,
+                   q_rank=1536, lin_heads=32, lin_dim=128, lin_vdim=128, inner=16, qk_heads=8, taps=4, ff=12288, experts=16, identity=2, top=4,
+                   groups=(4, 2), eff=3072, shared_ff=3072, side=0, times=1, vocab=32768),
+}
+
+
 def peaks(root: str) -> tuple[float, float, str]:
     p = os.path.join(root, "MEASURED_PEAKS.json")
     if os.path.exists(p):
@@ -307,6 +319,74 @@ def vosolorn_twin_bytes_flops(s: dict, T: int, B: int, ctx: int) -> tuple[float,
     dec = 2 * weights + B * (2 * 2 * G * D * seen + 2 * state) + 2 * s["vocab"] * W
     attn_fl = 2 * T * H * seen_avg * 2 * D + 2 * T * s["lin_heads"] * 4 * s["lin_dim"] * s["lin_vdim"]
     return float(dec), float(2 * T * weights + attn_fl + 2 * s["vocab"] * W)
+
+
+def goluzen_config(s: dict):
+    from pygpukit_b200.llm.config import layered_config_from_json
+    dense = {"kind": "dense", "ff": s["ff"]}
+    moe = {"kind": "moe", "expert": {"ff": s["eff"]}, "shared": {"ff": s["shared_ff"]},
+           "router": {"experts": s["experts"], "top": s["top"], "scale": 2.0, "groups": {"count": s["groups"][0], "keep": s["groups"][1]}}}
+    latent = {"heads": s["heads"], "dim": s["ldim"], "rot_dim": s["lrot"], "vdim": s["lvdim"], "kv_rank": s["kv_rank"],
+              "scale": (s["ldim"] + s["lrot"]) ** -0.5, "mask": {"size": s["window"]},
+              "rot": {"dims": s["lrot"], "base": 10000.0, "scaling": {"factor": 4.0, "original": 4096, "fast": 32.0, "slow": 1.0}}}
+    attention = {"heads": s["heads"], "kv_heads": s["kv_heads"], "dim": s["dim"], "vdim": s["dim"], "scale": s["dim"] ** -0.5, "softcap": 30.0,
+                 "mask": {"size": s["window"], "keep_first": s["keep"]}, "rot": {"dims": s["rot"], "base": 10000.0, "scaling": {"factor": 2.0}}}
+    gla = {"heads": s["lin_heads"], "dim": s["lin_dim"], "vdim": s["lin_vdim"], "tau": 16.0}
+    layers = [{"type": "latent_attention", "mlp": dense, "mixer": latent}, {"type": "gla", "mlp": moe, "mixer": gla},
+              {"type": "attention", "mlp": moe, "mixer": attention}, {"type": "latent_attention", "mlp": dense, "mixer": dict(latent, kv_from=0)}]
+    return layered_config_from_json({"architecture": "Goluzen", "layers": layers, "norm": {"eps": 1e-6}, "embedding": {"scale": 1.0},
+                                     "vocab": s["vocab"], "width": s["width"]})
+
+
+def goluzen_bytes_flops(s: dict, T: int, B: int, ctx: int) -> tuple[float, float]:
+    """(bytes a decode step of B tokens touches, FLOPs of a T-token prefill; the gated linear attention counted in its recurrent form,
+    the latent layers in their absorbed form)"""
+    W, H, G, D, V, win = s["width"], s["heads"], s["kv_heads"], s["dim"], s["vocab"], s["window"]
+    R, rot, Dl, Dlv = s["kv_rank"], s["lrot"], s["ldim"], s["lvdim"]
+    Hg, Dg, Dgv, r = s["lin_heads"], s["lin_dim"], s["lin_vdim"], s["inner"]
+    lat_w = (H * (Dl + rot) + H * Dlv) * W + H * (Dl + Dlv) * R + W * H * Dlv             # each of the two
+    dkv_w = (R + rot) * W
+    gla_w = (2 * Hg * Dg + 2 * Hg * Dgv + r) * W + W * Hg * Dgv
+    att_w = (H * D + 2 * G * D) * W + W * H * D
+    dense_w, exp_w, sh_w = 2 * s["ff"] * W, 2 * s["eff"] * W, 2 * s["shared_ff"] * W
+    act = min(s["experts"], B * s["top"])
+    router = (s["experts"] + 1) * W
+    state = 2 * 4 * Hg * Dg * Dgv
+    seen, seen_lat = min(ctx, win + s["keep"]), min(ctx, win)
+    weights = 2 * lat_w + dkv_w + gla_w + att_w + 2 * dense_w
+    dec = (2 * (weights + 2 * (sh_w + act * exp_w)) + 4 * (2 * router + r * Hg * Dg) + 2 * V * W
+           + B * (2 * 2 * G * D * seen + 2 * 2 * (R + rot) * seen_lat + state))
+    seen_avg = T / 2 if T <= win else win * (1 - win / (2 * T))
+    per_tok = weights + 2 * (router + sh_w + s["top"] * exp_w) + r * Hg * Dg
+    attn_fl = 2 * T * H * seen_avg * 2 * D + 2 * 2 * T * H * seen_avg * (2 * R + rot) + 2 * T * Hg * 2 * Dg * Dgv
+    return float(dec), float(2 * T * per_tok + attn_fl + 2 * V * W)
+
+
+def goluzen_turutar_twin(s: dict) -> dict:
+    """Turutar's sizes for the same heads and feed-forwards: a latent layer over the whole context and a windowed one, twice"""
+    return dict(s, rot=s["lrot"], times=2)
+
+
+def main_goluzen(root: str, sizes: list[str], steps: int, warm: int, prompt: int = 2000) -> dict:
+    """Goluzen beside the two closest existing models at equal sizes -- Sumitar (windowed attention, a gated recurrence with a state per
+    sequence, experts behind a router with a choice bias) and Turutar (latent and windowed attention): prefill of `prompt` tokens,
+    decode of 1 and 8 requests at that context."""
+    from pygpukit_b200._lib import api
+    hbm, tflops, src = peaks(root)
+    res = {"metric": "goluzen_prefill_decode_tokens_per_s", "data": "synthetic",
+           "dtype": "bf16 matrices and cache, f32 residual / norms / scores / router / decays / recurrent state",
+           "peaks": {"hbm_gbs": hbm, "bf16_tflops": tflops, "source": src}, "prompt": prompt, "steps": steps, "warmup": warm, "sizes": {}}
+    for name in sizes:
+        s = GOLUZEN_SIZES[name]
+        t = goluzen_turutar_twin(s)
+        entry = {"shape": {k: (list(v) if isinstance(v, tuple) else v) for k, v in s.items()}}
+        for key, cfg, count in (("goluzen", goluzen_config(s), lambda T, B, ctx: goluzen_bytes_flops(s, T, B, ctx)),
+                                ("sumitar_twin", sumitar_config(s), lambda T, B, ctx: sumitar_bytes_flops(s, T, B, ctx)),
+                                ("turutar_twin", turutar_config(t), lambda T, B, ctx: turutar_bytes_flops(t, T, B, ctx))):
+            entry[key] = run_layered(cfg, count, s["vocab"], prompt, (1, 8), steps, max(3, warm), hbm, tflops)
+            api.device_sync()
+        res["sizes"][name] = entry
+    return res
 
 
 def _timed(fn, iters: int, warm: int) -> float:
