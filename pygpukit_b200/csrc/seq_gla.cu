@@ -43,6 +43,12 @@ struct GlaArgs {
 __device__ __forceinline__ float silu_f(float z) { return z / (1.f + expf(-z)); }
 __device__ __forceinline__ float log_sigmoid(float z) { return fminf(z, 0.f) - log1pf(expf(-fabsf(z))); }
 constexpr float LOG2E = 1.44269504088896340736f;
+// 2^x for decays: numbers too small to be normal count as zero
+__device__ __forceinline__ float exp2_f(float x) {
+    float r;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(x));
+    return r;
+}
 
 // ---------------------------------------------------------------- one token per sequence
 constexpr int ST = 256;                 // threads per block
@@ -233,20 +239,22 @@ __device__ __forceinline__ size_t chunk_row(const ChunkArgs& c, int seq, int chu
     return (((size_t)seq * c.chunks + chunk) * c.a.H + h) * ((size_t)c.a.D * c.a.Dv + c.a.D);
 }
 
-// rows of `cols` columns at `src` into shared memory (row stride ls), zeros from row nc / column cols on
-template <int MC, int NT>
-__device__ __forceinline__ void stage_rows(const float* src, int ld, int nc, int cols, float* dst, int ls, bool vec) {
-    if (vec) {
-        const int c4 = ls >> 2;
-        for (int i = threadIdx.x; i < MC * c4; i += NT) {
-            const int r = i / c4, c = (i - r * c4) * 4;
-            if (r < nc && c < cols) cp_async16(dst + r * ls + c, src + (size_t)r * ld + c);
-            else *(float4*)(dst + r * ls + c) = make_float4(0.f, 0.f, 0.f, 0.f);
-        }
-    } else {
-        for (int i = threadIdx.x; i < MC * ls; i += NT) {
-            const int r = i / ls, c = i - r * ls;
-            dst[i] = (r < nc && c < cols) ? src[(size_t)r * ld + c] : 0.f;
+// ROWS rows of `cols` columns at `src` into shared memory (row stride ls, a multiple of 4) by asynchronous copies, zeros from row nc /
+// column cols on; a warp per row
+template <int ROWS, int NT>
+__device__ __forceinline__ void stage_rows(const float* src, size_t ld, int nc, int cols, float* dst, int ls, bool vec) {
+    const int lane = threadIdx.x & 31;
+    for (int r = threadIdx.x >> 5; r < ROWS; r += NT / 32) {
+        const float* s = src + (size_t)r * ld;
+        float* d = dst + r * ls;
+        if (vec) {
+            for (int c = lane * 4; c < ls; c += 128)
+                if (r < nc && c < cols) cp_async16(d + c, s + c);
+                else *(float4*)(d + c) = make_float4(0.f, 0.f, 0.f, 0.f);
+        } else {
+            for (int c = lane; c < ls; c += 32)
+                if (r < nc && c < cols) cp_async4(d + c, s + c);
+                else d[c] = 0.f;
         }
     }
 }
@@ -261,8 +269,9 @@ __global__ void __launch_bounds__(256) gla_update_kernel(ChunkArgs p) {
     const int cw = slice_cols(Dv, p.slices), v0 = sl * cw, nv = min(cw, Dv - v0);
     float* Ks = sm;                      // [MC][D8], decayed to the chunk's end
     float* Vs = Ks + MC * D8;            // [MC][cw]
+    float* Es = Vs + MC * cw;            // [NS][D8] sum of log2 decays from a sub-chunk's start to the chunk's end
     const int4 sq = a.seqs[blockIdx.y];
-    const int c = p.c_begin + blockIdx.x, tid = threadIdx.x;
+    const int c = p.c_begin + blockIdx.x, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     if (c * MC >= sq.y || nv <= 0) return;
     const int nc = min(MC, sq.y - c * MC), r0 = sq.x + c * MC;
     const size_t hd = (size_t)a.H * D;
@@ -270,34 +279,32 @@ __global__ void __launch_bounds__(256) gla_update_kernel(ChunkArgs p) {
     cp_async_commit();
     const float* Lh = p.L + (size_t)r0 * hd + (size_t)h * D;
     float* U = p.ws + chunk_row(p, blockIdx.y, blockIdx.x, h);
-    constexpr int B = 8;                                   // loads in flight per thread
-    for (int i0 = tid; i0 < MC * D8; i0 += 256 * B) {
-        float kk[B], ee[B];
+    for (int d = tid; d < D; d += 256) {
+        float tot[NS], e = 0.f;
 #pragma unroll
-        for (int b = 0; b < B; ++b) {
-            const int i = i0 + 256 * b, s = i / D8, d = i - s * D8;
-            kk[b] = 0.f; ee[b] = 0.f;
-            if (i >= MC * D8 || s >= nc || d >= D) continue;
-            kk[b] = a.proj[(size_t)(r0 + s) * a.ld + a.k_off + (size_t)h * D + d];
-            float e = -Lh[(size_t)s * hd + d];
+        for (int j = 0; j < NS; ++j) tot[j] = j * SUB < nc ? Lh[(size_t)min(nc - 1, j * SUB + SUB - 1) * hd + d] : 0.f;
 #pragma unroll
-            for (int j = 0; j < NS; ++j)
-                if (j >= s / SUB && j * SUB < nc) e += Lh[(size_t)min(nc - 1, j * SUB + SUB - 1) * hd + d];
-            ee[b] = e;
-        }
-#pragma unroll
-        for (int b = 0; b < B; ++b) {
-            const int i = i0 + 256 * b;
-            if (i < MC * D8) Ks[i] = kk[b] * exp2f(ee[b]);
-        }
+        for (int j = NS - 1; j >= 0; --j) { e += tot[j]; Es[j * D8 + d] = e; }
+        if (sl == 0) U[(size_t)D * Dv + d] = exp2_f(e);
     }
-    if (sl == 0)
-        for (int d = tid; d < D; d += 256) {
-            float e = 0.f;
+    __syncthreads();
+    constexpr int B = 8;                                   // rows in flight per thread
+    const float* kr = a.proj + (size_t)r0 * a.ld + a.k_off + (size_t)h * D;
+    for (int d = lane; d < D8; d += 32)
+        for (int s0 = warp; s0 < MC; s0 += 8 * B) {
+            float kk[B], ll[B];
 #pragma unroll
-            for (int j = 0; j < NS; ++j)
-                if (j * SUB < nc) e += Lh[(size_t)min(nc - 1, j * SUB + SUB - 1) * hd + d];
-            U[(size_t)D * Dv + d] = exp2f(e);
+            for (int b = 0; b < B; ++b) {
+                const int s = s0 + 8 * b;
+                const bool in = s < nc && d < D;
+                kk[b] = in ? kr[(size_t)s * a.ld + d] : 0.f;
+                ll[b] = in ? Lh[(size_t)s * hd + d] : 0.f;
+            }
+#pragma unroll
+            for (int b = 0; b < B; ++b) {
+                const int s = s0 + 8 * b;
+                if (s < MC) Ks[s * D8 + d] = s < nc && d < D ? kk[b] * exp2_f(Es[(s / SUB) * D8 + d] - ll[b]) : 0.f;
+            }
         }
     cp_async_wait<0>();
     __syncthreads();
@@ -364,44 +371,53 @@ __global__ void __launch_bounds__(256) gla_scan_kernel(ChunkArgs p) {
 // outputs of a chunk
 constexpr int SLAB = 16;                 // state rows per slab
 
-// rows transposed into [D][MP]: a warp moves 8 consecutive elements of 4 rows at a time (whole sectors, no bank conflicts).  PAD:
-// rows behind the last one repeat it inside its sub-chunk (running sums); otherwise they are zero.
+// A [D][MC] tile whose rows are permuted in groups of four elements, so that transposing stores and the products' loads (four
+// neighbouring tokens of one channel, or sixteen of a channel and sixteen of the fourth one behind it) meet no bank conflicts
+template <int MC> __device__ __forceinline__ int at_dt(int d, int t) {
+    constexpr int M = MC / 4 < 8 ? MC / 4 - 1 : 7;
+    return d * MC + (t ^ ((d & M) << 2));
+}
+// Weights of a chunk: one [SUB keys][SUB queries] block per pair of sub-chunks i >= j
+__device__ __forceinline__ int at_st(int s, int t) {
+    const int i = t / SUB, j = s / SUB;
+    return ((i * (i + 1) / 2 + j) * SUB + s % SUB) * SUB + t % SUB;
+}
+
+// rows transposed into [D][MC]: a warp moves 8 consecutive elements of 4 rows at a time (whole sectors).  PAD: rows behind the last
+// one repeat it inside its sub-chunk (running sums); otherwise they are zero.
 template <int MC, int NT, bool PAD>
 __device__ __forceinline__ void stage_transposed(const float* src, size_t ld, int nc, int D, float mult, float* dst) {
-    constexpr int MP = MC + 4, B = 8, NW = NT / 32;
+    constexpr int B = 8, NW = NT / 32;
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, dl = lane & 7, tl = lane >> 3;
-    const int nd = (D + 7) / 8, last = (nc - 1) / SUB;
-    for (int u0 = warp; u0 < nd * (MC / 4); u0 += NW * B) {
-        float r[B];
+    const int last = (nc - 1) / SUB;
+    for (int tg = warp; tg < MC / 4; tg += NW) {
+        const int t = tg * 4 + tl;
+        const bool in = t < nc || (PAD && t / SUB == last);
+        const float* row = src + (size_t)min(t, nc - 1) * ld;
+        for (int d0 = dl; d0 < D; d0 += 8 * B) {
+            float r[B];
 #pragma unroll
-        for (int b = 0; b < B; ++b) {
-            const int u = u0 + NW * b, d = (u % nd) * 8 + dl, t = (u / nd) * 4 + tl;
-            const bool in = t < nc || (PAD && t / SUB == last);
-            r[b] = (d < D && t < MC && in) ? __ldg(src + (size_t)min(t, nc - 1) * ld + d) : 0.f;
-        }
+            for (int b = 0; b < B; ++b) r[b] = (in && d0 + 8 * b < D) ? __ldg(row + d0 + 8 * b) : 0.f;
 #pragma unroll
-        for (int b = 0; b < B; ++b) {
-            const int u = u0 + NW * b, d = (u % nd) * 8 + dl, t = (u / nd) * 4 + tl;
-            if (d < D && t < MC) dst[d * MP + t] = r[b] * mult;
+            for (int b = 0; b < B; ++b)
+                if (d0 + 8 * b < D) dst[at_dt<MC>(d0 + 8 * b, t)] = r[b] * mult;
         }
     }
 }
 
 template <int MC>
-__global__ void __launch_bounds__(8 * MC) gla_output_kernel(ChunkArgs p) {
+__global__ void __launch_bounds__(8 * MC, MC == 64 ? 2 : 1) gla_output_kernel(ChunkArgs p) {
     extern __shared__ __align__(16) float sm[];
-    constexpr int NT = 8 * MC, MP = MC + 4, NS = MC / SUB, NP = NS * (NS - 1) / 2;
+    constexpr int NT = 8 * MC, NS = MC / SUB, NP = NS * (NS - 1) / 2;
     const GlaArgs& a = p.a;
     const int D = a.D, Dv = a.Dv;
     const int h = blockIdx.z / p.slices, sl = blockIdx.z - h * p.slices;
     const int cw = slice_cols(Dv, p.slices), v0 = sl * cw, nv = min(cw, Dv - v0);
-    const int r1 = max(D * MP, MC * cw);
-    float* Qt = sm;                      // [D][MP]
-    float* R1 = Qt + D * MP;             // K transposed [D][MP], then V [MC][cw], then the outputs [MC][cw]
-    float* Lt = R1 + r1;                 // [D][MP] running sums of log2 decays
-    float* At = Lt + D * MP;             // [MC][MP]: weight of key s for query t at [s][t]
-    float* slab = At + MC * MP;          // [2][SLAB][cw]
-    float* Mb = slab + 2 * SLAB * cw;    // [NP][D] decays over the sub-chunks between two
+    float* Qt = sm;                      // [D][MC]
+    float* R1 = Qt + D * MC;             // K transposed [D][MC], then V [MC][cw], then the outputs [MC][cw]
+    float* Lt = R1 + MC * max(D, cw);    // [D][MC] running sums of log2 decays, then two slabs [SLAB][cw] of the starting state
+    float* At = Lt + max(D * MC, 2 * SLAB * cw);           // [NP + NS][SUB][SUB]: weight of key s for query t
+    float* Mb = At + (NP + NS) * SUB * SUB;                // [NP][D] decays over the sub-chunks between two
     const int4 sq = a.seqs[blockIdx.y];
     const int c = p.c_begin + blockIdx.x, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     if (c * MC >= sq.y || nv <= 0) return;
@@ -410,33 +426,18 @@ __global__ void __launch_bounds__(8 * MC) gla_output_kernel(ChunkArgs p) {
     const float* Sc = p.ws + chunk_row(p, blockIdx.y, blockIdx.x, h);
     const bool sv = a.vec && (D & 3) == 0;
     auto fetch_slab = [&](int b) {                         // slab b of the starting state
-        float* dst = slab + (b & 1) * SLAB * cw;
-        const int d0 = b * SLAB, rows = min(SLAB, D - d0);
-        if (sv) {
-            const int c4 = cw >> 2;
-            for (int i = tid; i < SLAB * c4; i += NT) {
-                const int r = i / c4, cc = (i - r * c4) * 4;
-                if (r < rows && cc < nv) cp_async16(dst + r * cw + cc, Sc + (size_t)(d0 + r) * Dv + v0 + cc);
-                else *(float4*)(dst + r * cw + cc) = make_float4(0.f, 0.f, 0.f, 0.f);
-            }
-        } else {
-            for (int i = tid; i < SLAB * cw; i += NT) {
-                const int r = i / cw, cc = i - r * cw;
-                if (r < rows && cc < nv) cp_async4(dst + i, Sc + (size_t)(d0 + r) * Dv + v0 + cc);
-                else dst[i] = 0.f;
-            }
-        }
+        stage_rows<SLAB, NT>(Sc + (size_t)b * SLAB * Dv + v0, Dv, min(SLAB, D - b * SLAB), nv, Lt + (b & 1) * SLAB * cw, cw, sv);
         cp_async_commit();
     };
-    if (has_state) fetch_slab(0);
     const float* rows = a.proj + (size_t)r0 * a.ld;
     const size_t hd = (size_t)a.H * D;
     stage_transposed<MC, NT, false>(rows + a.q_off + (size_t)h * D, a.ld, nc, D, a.q_scale, Qt);
     stage_transposed<MC, NT, false>(rows + a.k_off + (size_t)h * D, a.ld, nc, D, 1.f, R1);
     stage_transposed<MC, NT, true>(p.L + (size_t)r0 * hd + (size_t)h * D, hd, nc, D, 1.f, Lt);
-    for (int i = tid; i < MC * MP; i += NT) At[i] = 0.f;
+    for (int i = tid; i < (NP + NS) * SUB * SUB; i += NT) At[i] = 0.f;
     __syncthreads();
-    {   // weights inside a sub-chunk: four warps each, a warp takes four queries, a lane one key and every other group of four channels
+    {   // weights inside a sub-chunk: four warps each, a warp takes four queries, a lane one key and every other group of four channels.
+        // A key behind its query would give a positive exponent: such a pair's sum is thrown away.
         const int i = warp >> 2, tl = (warp & 3) * 4, s = lane & 15, half = lane >> 4;
         if (i * SUB + tl < nc) {
             const int t0 = i * SUB + tl, s0 = i * SUB + s;
@@ -446,35 +447,36 @@ __global__ void __launch_bounds__(8 * MC) gla_output_kernel(ChunkArgs p) {
                 for (int e = 0; e < 4; ++e) {
                     const int d = d0 + e;
                     if (d >= D) break;
-                    const float k = R1[d * MP + s0], l = Lt[d * MP + s0];
-                    const float4 q4 = *(const float4*)(Qt + d * MP + t0), l4 = *(const float4*)(Lt + d * MP + t0);
-                    acc[0] = fmaf(q4.x * k, exp2f(fminf(l4.x - l, 0.f)), acc[0]);
-                    acc[1] = fmaf(q4.y * k, exp2f(fminf(l4.y - l, 0.f)), acc[1]);
-                    acc[2] = fmaf(q4.z * k, exp2f(fminf(l4.z - l, 0.f)), acc[2]);
-                    acc[3] = fmaf(q4.w * k, exp2f(fminf(l4.w - l, 0.f)), acc[3]);
+                    const float k = R1[at_dt<MC>(d, s0)], l = Lt[at_dt<MC>(d, s0)];
+                    const float4 q4 = *(const float4*)(Qt + at_dt<MC>(d, t0)), l4 = *(const float4*)(Lt + at_dt<MC>(d, t0));
+                    acc[0] = fmaf(q4.x * k, exp2_f(l4.x - l), acc[0]);
+                    acc[1] = fmaf(q4.y * k, exp2_f(l4.y - l), acc[1]);
+                    acc[2] = fmaf(q4.z * k, exp2_f(l4.z - l), acc[2]);
+                    acc[3] = fmaf(q4.w * k, exp2_f(l4.w - l), acc[3]);
                 }
             }
 #pragma unroll
             for (int e = 0; e < 4; ++e) {
                 const float v = acc[e] + __shfl_xor_sync(0xffffffffu, acc[e], 16);
-                if (half == 0 && s <= tl + e && t0 + e < nc) At[s0 * MP + t0 + e] = v;
+                if (half == 0 && s <= tl + e && t0 + e < nc) At[at_st(s0, t0 + e)] = v;
             }
         }
     }
-    for (int i = tid; i < NP * D; i += NT) {               // pair (i, j), i > j, at i (i - 1) / 2 + j
-        const int pr = i / D, d = i - pr * D;
+    for (int pr = 0; pr < NP; ++pr) {                      // pair (i, j), i > j, at i (i - 1) / 2 + j
         int hi = 1, lo = pr;
         while (lo >= hi) { lo -= hi; ++hi; }
-        float e = 0.f;
-        for (int m = lo + 1; m < hi; ++m) e += Lt[d * MP + m * SUB + SUB - 1];
-        Mb[i] = exp2f(e);
+        for (int d = tid; d < D; d += NT) {
+            float e = 0.f;
+            for (int m = lo + 1; m < hi; ++m) e += Lt[at_dt<MC>(d, m * SUB + SUB - 1)];
+            Mb[pr * D + d] = exp2_f(e);
+        }
     }
     __syncthreads();
     for (int i = tid; i < D * MC; i += NT) {               // q decayed from its sub-chunk's start, k to its sub-chunk's end
-        const int d = i / MC, t = i - d * MC;
-        const float l = Lt[d * MP + t];
-        Qt[d * MP + t] *= exp2f(l);
-        R1[d * MP + t] *= exp2f(Lt[d * MP + (t / SUB) * SUB + SUB - 1] - l);
+        const int d = i / MC, t = i - d * MC, o = at_dt<MC>(d, t);
+        const float l = Lt[o];
+        Qt[o] *= exp2_f(l);
+        R1[o] *= exp2_f(Lt[at_dt<MC>(d, (t / SUB) * SUB + SUB - 1)] - l);
     }
     __syncthreads();
     if (NP > 0) {   // weights between sub-chunks: 64 threads per pair, 2 queries x 2 keys each
@@ -486,28 +488,32 @@ __global__ void __launch_bounds__(8 * MC) gla_output_kernel(ChunkArgs p) {
             if (t0 >= nc) continue;
             float a00 = 0.f, a01 = 0.f, a10 = 0.f, a11 = 0.f;
             const float* mp = Mb + pr * D;
-#pragma unroll 4
+#pragma unroll 8
             for (int d = 0; d < D; ++d) {
-                const float2 q2 = *(const float2*)(Qt + d * MP + t0), k2 = *(const float2*)(R1 + d * MP + s0);
+                const float2 q2 = *(const float2*)(Qt + at_dt<MC>(d, t0)), k2 = *(const float2*)(R1 + at_dt<MC>(d, s0));
                 const float m = mp[d], kx = k2.x * m, ky = k2.y * m;
                 a00 = fmaf(q2.x, kx, a00); a01 = fmaf(q2.x, ky, a01);
                 a10 = fmaf(q2.y, kx, a10); a11 = fmaf(q2.y, ky, a11);
             }
-            *(float2*)(At + s0 * MP + t0) = make_float2(a00, a10);
-            *(float2*)(At + (s0 + 1) * MP + t0) = make_float2(a01, a11);
+            *(float2*)(At + at_st(s0, t0)) = make_float2(a00, a10);
+            *(float2*)(At + at_st(s0 + 1, t0)) = make_float2(a01, a11);
         }
     }
     __syncthreads();                                       // K is done: V takes its place
     stage_rows<MC, NT>(rows + a.v_off + (size_t)h * Dv + v0, a.ld, nc, nv, R1, cw, a.vec);
     cp_async_commit();
-    if (NS > 1 && has_state)                               // q decayed from the chunk's start
-        for (int i = tid; i < D * MC; i += NT) {
-            const int d = i / MC, t = i - d * MC;
-            if (t < SUB) continue;
-            float e = 0.f;
-            for (int m = 0; m < t / SUB; ++m) e += Lt[d * MP + m * SUB + SUB - 1];
-            Qt[d * MP + t] *= exp2f(e);
-        }
+    if (has_state) {
+        if (NS > 1)                                        // q decayed from the chunk's start
+            for (int i = tid; i < D * MC; i += NT) {
+                const int d = i / MC, t = i - d * MC;
+                if (t < SUB) continue;
+                float e = 0.f;
+                for (int m = 0; m < t / SUB; ++m) e += Lt[at_dt<MC>(d, m * SUB + SUB - 1)];
+                Qt[at_dt<MC>(d, t)] *= exp2_f(e);
+            }
+        __syncthreads();                                   // the running sums are done: the state's slabs take their place
+        fetch_slab(0);
+    }
     const int nTv = cw / 4, ntiles = (MC / 4) * nTv;       // at most NT tiles of 4 tokens x 4 value columns
     const bool live = tid < ntiles;
     const int t0 = live ? (tid / nTv) * 4 : 0, w0 = live ? (tid % nTv) * 4 : 0;
@@ -525,11 +531,11 @@ __global__ void __launch_bounds__(8 * MC) gla_output_kernel(ChunkArgs p) {
             }
             if (b > 0) __syncthreads();
             if (live) {
-                const float* sb = slab + (b & 1) * SLAB * cw + w0;
+                const float* sb = Lt + (b & 1) * SLAB * cw + w0;
                 const int ndd = min(SLAB, D - b * SLAB);
-#pragma unroll 4
+#pragma unroll 8
                 for (int d = 0; d < ndd; ++d) {
-                    const float4 q4 = *(const float4*)(Qt + (b * SLAB + d) * MP + t0), s4 = *(const float4*)(sb + d * cw);
+                    const float4 q4 = *(const float4*)(Qt + at_dt<MC>(b * SLAB + d, t0)), s4 = *(const float4*)(sb + d * cw);
                     const float qq[4] = {q4.x, q4.y, q4.z, q4.w}, ssv[4] = {s4.x, s4.y, s4.z, s4.w};
 #pragma unroll
                     for (int i = 0; i < 4; ++i)
@@ -542,14 +548,19 @@ __global__ void __launch_bounds__(8 * MC) gla_output_kernel(ChunkArgs p) {
     }
     if (live) {
         const int send = min(nc, t0 + 4);
+        const float* ar = At + at_st(0, t0);
+        for (int j = 0; j * SUB < send; ++j) {             // one block of weights after the other
+            const int ns = min(SUB, send - j * SUB);
+            const float* vr = R1 + j * SUB * cw + w0;
 #pragma unroll 4
-        for (int s = 0; s < send; ++s) {
-            const float4 aa = *(const float4*)(At + s * MP + t0), v4 = *(const float4*)(R1 + s * cw + w0);
-            const float ww[4] = {aa.x, aa.y, aa.z, aa.w}, vv[4] = {v4.x, v4.y, v4.z, v4.w};
+            for (int s = 0; s < ns; ++s) {
+                const float4 aa = *(const float4*)(ar + (j * SUB + s) * SUB), v4 = *(const float4*)(vr + s * cw);
+                const float ww[4] = {aa.x, aa.y, aa.z, aa.w}, vv[4] = {v4.x, v4.y, v4.z, v4.w};
 #pragma unroll
-            for (int i = 0; i < 4; ++i)
+                for (int i = 0; i < 4; ++i)
 #pragma unroll
-                for (int j = 0; j < 4; ++j) acc[i][j] = fmaf(ww[i], vv[j], acc[i][j]);
+                    for (int k = 0; k < 4; ++k) acc[i][k] = fmaf(ww[i], vv[k], acc[i][k]);
+            }
         }
     }
     __syncthreads();                                       // V is done: the outputs take its place
@@ -602,8 +613,8 @@ int launch_step(const GlaArgs& a, int n_seqs, int blocks, int slice, cudaStream_
 constexpr size_t CHUNK_SMEM = 224 * 1024;
 
 size_t output_smem(int MC, int D, int cw) {
-    const size_t MP = MC + 4, ns = MC / SUB, r1 = D * MP > (size_t)MC * cw ? D * MP : (size_t)MC * cw;
-    return sizeof(float) * (2 * D * MP + r1 + MC * MP + 2 * (size_t)SLAB * cw + ns * (ns - 1) / 2 * D);
+    const size_t ns = MC / SUB, np = ns * (ns - 1) / 2, dm = (size_t)D * MC, vm = (size_t)MC * cw, sl = 2 * (size_t)SLAB * cw;
+    return sizeof(float) * (dm + (dm > vm ? dm : vm) + (dm > sl ? dm : sl) + (np + ns) * SUB * SUB + np * D);
 }
 int value_slices(int vdim) { return (vdim + SLICE_MAX - 1) / SLICE_MAX; }
 // tokens per chunk: what fits a block's shared memory (0: keys too large)
@@ -618,7 +629,7 @@ template <int MC>
 int launch_chunks(ChunkArgs& p, int n_seqs, cudaStream_t st) {
     const GlaArgs& a = p.a;
     const int cw = slice_cols(a.Dv, p.slices), D8 = (a.D + 7) & ~7;
-    const size_t smem_u = sizeof(float) * ((size_t)MC * D8 + (size_t)MC * cw), smem_o = output_smem(MC, a.D, cw);
+    const size_t smem_u = sizeof(float) * ((size_t)MC * D8 + (size_t)MC * cw + (size_t)(MC / SUB) * D8), smem_o = output_smem(MC, a.D, cw);
     static bool configured = false;
     if (!configured) {
         PGK_CUDA(cudaFuncSetAttribute(gla_update_kernel<MC>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)CHUNK_SMEM));

@@ -219,7 +219,7 @@ class DecayHarness:
 # key sizes that fill chunks of 64, 32 and 16 tokens, values of one column, of one block and of several
 DECAY_LAYOUTS = [dict(H=3, D=8, Dv=6), dict(H=1, D=44, Dv=60, tau=16.0, pad=3), dict(H=2, D=70, Dv=9, inner=1), dict(H=2, D=130, Dv=20, tau=1.0),
                  dict(H=5, D=16, Dv=33, inner=40), dict(H=2, D=20, Dv=260), dict(H=1, D=12, Dv=1030), dict(H=4, D=64, Dv=128, inner=16),
-                 dict(H=2, D=1, Dv=1), dict(H=1, D=300, Dv=12, tau=30.0), dict(H=1, D=520, Dv=8, inner=3)]
+                 dict(H=2, D=1, Dv=1), dict(H=1, D=300, Dv=12, tau=30.0), dict(H=1, D=600, Dv=8, inner=3)]
 
 
 @pytest.mark.parametrize("layout", DECAY_LAYOUTS)
@@ -235,7 +235,7 @@ def test_gated_linear_attention_whole_portions_and_single_tokens_agree_with_the_
 
 
 def test_chunk_sizes_follow_the_key_size():
-    assert [api.seq_gla_chunk_tokens(D, 64) for D in (16, 128, 300, 520)] == [64, 64, 32, 16]
+    assert [api.seq_gla_chunk_tokens(D, 64) for D in (16, 128, 300, 600)] == [64, 64, 32, 16]
     assert api.seq_gla_chunk_tokens(5000, 64) == 0
 
 
